@@ -99,8 +99,10 @@ class ModelRunner:
         # that reaches max_seq_len keeps generating over its most recent tokens; the cache evicts whole blocks from the
         # front (block table shifted left, block returned to the pool) and positions stay absolute, which rotary
         # embeddings allow (keys keep the rotation of the position they were written at).  Families with a learned
-        # position table cannot index past it, so they keep stopping at max_seq_len.
-        self.sliding = bool(sliding_window) and not self.spec.learned_pos and not self.recurrent
+        # position table cannot index past it, so they keep stopping at max_seq_len.  So do models whose attention goes by
+        # the place of a key in the sequence (first tokens that a window keeps): eviction would renumber the keys.
+        self.sliding = (bool(sliding_window) and not self.spec.learned_pos and not self.recurrent
+                        and not getattr(core, "needs_first_pages", False))
         self.block_size = block_size
         self.max_blocks_per_seq = -(-self.max_seq_len // block_size)
         if num_blocks is None and pool_tokens:

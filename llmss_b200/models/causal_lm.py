@@ -21,6 +21,7 @@ from .botalorn import BotalornLM, botalorn_spec, load_botalorn
 from .decoder import DecoderLM
 from .families import FAMILIES
 from .ninelix import NinelixLM, load_ninelix, ninelix_spec
+from .rofulorn import RofulornLM, load_rofulorn, rofulorn_spec
 from .zenorax import ZenoraxLM, load_zenorax, zenorax_spec
 
 
@@ -181,6 +182,21 @@ class ZenoraxForCausalLM(CausalLM):
         self.core.finalize()
 
 
+class RofulornForCausalLM(CausalLM):
+    """Native architecture (see models/rofulorn.py): parallel sub-layers over a 32-bit residual stream, differential and plain
+    windowed rotary attention, layers that share keys and values, gated feed-forward.  Same constructor and forward interface as
+    the HF-shaped classes."""
+    family = "rofulorn"
+    float32_on_cuda = True
+
+    def __init__(self, config, weights, fuse_parallel: bool = True):
+        nn.Module.__init__(self)
+        self.config = config
+        self.core = RofulornLM(rofulorn_spec(config), weights.process_group, weights.device, weights.dtype)
+        load_rofulorn(self.core, weights)
+        self.core.finalize()
+
+
 MODEL_REGISTRY = {
     "gptj": GPTJForCausalLM,
     "gpt_bigcode": GPTBigCodeForCausalLM,
@@ -191,4 +207,5 @@ MODEL_REGISTRY = {
     "ninelix": NinelixForCausalLM,
     "botalorn": BotalornForCausalLM,
     "zenorax": ZenoraxForCausalLM,
+    "rofulorn": RofulornForCausalLM,
 }

@@ -12,10 +12,14 @@
     layer may attend over the pages another layer writes;
   * ``SinkAttention`` -- grouped-query softmax attention whose values are the projected keys, with rotary positions from
     a frequency table, unit-RMS queries / keys and a learned sink logit per head in the softmax denominator;
+  * ``RotaryAttention`` -- grouped-query softmax attention with rotary positions from a frequency table, an optional query /
+    key norm per head, a sliding window that may keep the first tokens, soft-capped scores, optionally two maps per head that
+    are subtracted (differential attention); a layer may attend over the pages another layer writes;
   * ``Hgrn2Mixer`` -- a gated linear recurrence whose forget gate (bounded from below) also sets the write strength;
   * ``DeltaMixer`` -- the gated delta rule (ops.delta_scan) behind short convolutions, with a gated per-head norm;
   * ``HyperConnection`` -- the read / mix / write weights of one sub-layer over several residual streams;
-  * ``DenseFFN``.
+  * ``DenseFFN``, ``GatedFFN``;
+  * ``ParallelBlock`` -- a mixer and a feed-forward that read the same normed input and are summed, with one output product.
 
 Every block says what it keeps per sequence (``state_shapes``), which cache pages it needs (``kv_shape``), and maps
 (x: the 32-bit residual, h: x in the compute type) to a 32-bit [T, width] output.  All sizes and constants are
@@ -29,9 +33,10 @@ import math
 import torch
 
 from .. import ops
-from ..ops import (ACT_GELU_ERF, ACT_NONE, ACT_SILU, DECAY_HEAD, DECAY_TOKEN_CHANNEL, DECAY_TOKEN_HEAD, GATE_NONE, GATE_SIGMOID,
+from ..ops import (ACT_GELU_ERF, ACT_GELU_TANH, ACT_NONE, ACT_SILU, DECAY_HEAD, DECAY_TOKEN_CHANNEL, DECAY_TOKEN_HEAD, GATE_NONE, GATE_SIGMOID,
                    GATE_SILU, UNARY_NEG_EXP, UNARY_TANH)
 from ..utils.tracing import trace
+from .decoder import interleave_gate_up
 
 F32 = torch.float32
 
@@ -421,6 +426,80 @@ class SinkAttention:
             return ops.linear(ctx, self.w_o, out_dtype=F32)
 
 
+class RotaryAttention:
+    """Grouped-query softmax attention with rotary positions from a frequency table (ops.rotary_frequencies).
+
+        q, k, v = W h (+ b)  ->  q, k: per head and map rms_div * weight (if ``set_weights`` got norm weights), then rotation
+        s_ij = scale * q_i . k_j ;  s <- softcap * tanh(s / softcap)                              (softcap 0: no cap)
+        i sees j <= i with i - j < window or j < keep_first                                       (window 0: every j <= i)
+        plain:         o_h = softmax(s) v
+        differential:  two maps of size dim per head over one value,  o_h = rms_div(a_1 - lam a_2) * (1 - diff),
+                       lam = exp(lq1 . lk1) - exp(lq2 . lk2) + diff                               (one number per layer)
+        out = W_o concat_h(o) (+ b)
+
+    Cached: normed and rotated keys (both maps of a head in one row of its K page) and the projected values.  ``kv_from`` =
+    key of another layer: this layer has no key / value tensors and attends over that layer's pages with its own queries, mask
+    and combination.  One input GEMM over the stacked rows [q | k | v]."""
+
+    def __init__(self, width, heads, kv_heads, dim, vdim, scale, eps, freq, mag=1.0, interleaved=True, window=0, keep_first=0,
+                 softcap=0.0, diff=None, kv_from=None):
+        self.width, self.heads, self.kv_heads, self.dim, self.vdim, self.scale, self.eps = width, heads, kv_heads, dim, vdim, scale, eps
+        self.freq, self.mag, self.interleaved = freq, mag, interleaved
+        self.window, self.keep_first, self.softcap = int(window or 0), int(keep_first or 0), float(softcap or 0.0)
+        self.diff, self.maps, self.kv_from, self.own_kv = diff, (1 if diff is None else 2), kv_from, kv_from is None
+        assert heads % kv_heads == 0, "rotary attention: query heads must be a multiple of key/value heads"
+        assert 2 * freq.numel() <= dim, "rotary attention: more rotated channels than the head has"
+        self.w_in = self.b_in = self.q_norm = self.k_norm = self.w_o = self.b_o = None
+        self.combine = None          # (lam, eps, 1 - diff) of the differential form
+
+    @property
+    def n_out(self) -> int:
+        return self.heads * self.vdim
+
+    def state_shapes(self):
+        return {}
+
+    def kv_shape(self):
+        return (self.kv_heads, self.maps * self.dim, self.vdim) if self.own_kv else None
+
+    def weights(self):
+        return [self.w_in, self.b_in, self.q_norm, self.k_norm, self.w_o, self.b_o]
+
+    def set_weights(self, wq, wk, wv, w_o, bq=None, bk=None, bv=None, b_o=None, q_norm=None, k_norm=None, lam_vectors=None):
+        """wk / wv / bk / bv / k_norm are None for a layer that borrows its keys and values; ``lam_vectors``: (lq1, lk1, lq2, lk2)."""
+        ws = [wq, wk, wv] if self.own_kv else [wq]
+        bs = [bq, bk, bv] if self.own_kv else [bq]
+        self.w_in = torch.cat(ws, dim=0).contiguous()
+        if any(b is not None for b in bs):
+            self.b_in = torch.cat([b if b is not None else torch.zeros(w.shape[0], dtype=w.dtype, device=w.device)
+                                   for b, w in zip(bs, ws)]).contiguous()
+        self.q_norm, self.k_norm, self.w_o, self.b_o = q_norm, k_norm, w_o.contiguous(), b_o
+        self.freq = self.freq.to(torch.float64).to(w_o.device).contiguous()     # the kernels read the table on the device
+        if self.diff is not None:
+            lq1, lk1, lq2, lk2 = (t.double().cpu() for t in lam_vectors)
+            lam = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum())) + self.diff
+            self.combine = (lam, self.eps, 1.0 - self.diff)
+
+    def context(self, h, batch, lc, dtype, out=None):
+        """The concatenated heads [T, heads * vdim] in front of W_o (into ``out`` if given); ``lc``: this layer's cache view, whose
+        pages are the lender's when keys and values are borrowed."""
+        H, G, D, Dv = self.heads, self.kv_heads, self.dim, self.vdim
+        with trace("gemm_in"):
+            y = ops.linear(h, self.w_in, self.b_in, out_dtype=F32)
+        with trace("norm_rope_kv_write"):
+            q = ops.norm_rope_kv_write(y, H, G if self.own_kv else 0, D, Dv, self.maps, self.q_norm, self.k_norm, self.eps, self.freq,
+                                       self.mag, self.interleaved, batch.positions, batch.slot_mapping, lc.k, lc.v, batch=batch,
+                                       out_dtype=dtype)
+        with trace("attention_window" if self.diff is None else "attention_diff"):
+            return ops.attention_bias(q, lc.k, lc.v, batch, H, G, D, Dv, self.scale, None, out_dtype=dtype, window=self.window,
+                                      keep_first=self.keep_first, softcap=self.softcap, diff=self.combine, out=out)
+
+    def forward(self, h, batch, lc, dtype):
+        ctx = self.context(h, batch, lc, dtype)
+        with trace("gemm_out"):
+            return ops.linear(ctx, self.w_o, self.b_o, out_dtype=F32)
+
+
 class Hgrn2Mixer:
     """Gated linear recurrence in which the forget gate also decides what is written (HGRN2).
 
@@ -556,3 +635,64 @@ class DenseFFN:
             a = ops.linear(h, self.w_up, act=self.act)
         with trace("ffn_down"):
             return ops.linear(a, self.w_down, out_dtype=F32)
+
+
+class GatedFFN:
+    """W_down (act(W_gate h) * (W_up h)); gate and up rows interleave in one GEMM whose epilogue forms the product."""
+
+    def __init__(self, act: int = ACT_GELU_TANH):
+        self.act = act
+        self.w_gu = self.w_down = None
+
+    @property
+    def n_out(self) -> int:
+        return self.w_down.shape[1]
+
+    def weights(self):
+        return [self.w_gu, self.w_down]
+
+    def set_weights(self, w_gate, w_up, w_down):
+        self.w_gu, self.w_down = interleave_gate_up(w_gate, w_up), w_down.contiguous()
+
+    def hidden(self, h, out=None):
+        with trace("ffn_up"):
+            return ops.linear(h, self.w_gu, act=self.act, gated=True, out=out)
+
+    def forward(self, h):
+        a = self.hidden(h)
+        with trace("ffn_down"):
+            return ops.linear(a, self.w_down, out_dtype=F32)
+
+
+class ParallelBlock:
+    """mixer(h) + ffn(h) as one sub-layer: W_o and W_down lie side by side, the mixer's heads and the feed-forward's hidden row
+    are written side by side, and one GEMM forms the sum of both outputs in 32-bit.  ``ffn`` None: the mixer alone.  The mixer
+    offers ``context(h, batch, lc, dtype, out)`` / ``n_out`` / ``w_o`` / ``b_o`` and the feed-forward ``hidden(h, out)`` / ``n_out`` /
+    ``w_down``."""
+
+    def __init__(self, mixer, ffn=None):
+        self.mixer, self.ffn = mixer, ffn
+        self.w_out = None
+
+    def weights(self):
+        """Both output matrices live in ``w_out`` after ``finalize``."""
+        m = [t for t in self.mixer.weights() if t is not self.mixer.w_o]
+        f = [t for t in self.ffn.weights() if t is not self.ffn.w_down] if self.ffn is not None else []
+        return m + f + [self.w_out]
+
+    def finalize(self):
+        mx, ff = self.mixer, self.ffn
+        self.n_ctx, self.n_cat = mx.n_out, mx.n_out + (ff.n_out if ff is not None else 0)
+        self.w_out = torch.cat([mx.w_o, ff.w_down], dim=1).contiguous() if ff is not None else mx.w_o
+        mx.w_o = self.w_out[:, :self.n_ctx]
+        if ff is not None:
+            ff.w_down = self.w_out[:, self.n_ctx:]
+
+    def forward(self, h, batch, lc, dtype):
+        T = h.shape[0]
+        cat = torch.empty(T, self.n_cat, dtype=dtype, device=h.device)
+        self.mixer.context(h, batch, lc, dtype, out=cat[:, :self.n_ctx])
+        if self.ffn is not None:
+            self.ffn.hidden(h, out=cat[:, self.n_ctx:])
+        with trace("gemm_out"):
+            return ops.linear(cat, self.w_out, self.mixer.b_o, out_dtype=F32)

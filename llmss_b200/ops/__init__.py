@@ -64,8 +64,8 @@ def _fused_ar_mode(cu, symm, M: int, N: int, K: int, esz: int) -> int:
 
 
 def linear(x, w, bias=None, act: int = ACT_NONE, gated: bool = False, act_start: int = 0, residual=None,
-           out_dtype=None, comm=None):
-    """y = epilogue(x @ w.T); with ``comm`` the product is summed over the TP group first
+           out_dtype=None, comm=None, out=None):
+    """y = epilogue(x @ w.T) (into ``out``, e.g. columns of another product's operand, if given); with ``comm`` the product is summed over the TP group first
     (row-parallel layer: reference `TensorParallelRowLinear.forward`, layers.py:175-179) and
     bias/residual are applied once after the reduction."""
     reduce = comm is not None and not comm.single
@@ -73,7 +73,8 @@ def linear(x, w, bias=None, act: int = ACT_NONE, gated: bool = False, act_start:
         from . import cuda_impl as cu
 
         if not reduce:
-            return cu.linear(x, w, bias, act, gated, act_start, residual, out_dtype)
+            return cu.linear(x, w, bias, act, gated, act_start, residual, out_dtype, out=out)
+        assert out is None, "linear: out belongs to the unreduced form"
         symm = comm.symm
         if symm is not None:
             mode = _fused_ar_mode(cu, symm, x.shape[0], w.shape[0], x.shape[1], x.element_size())
@@ -87,7 +88,8 @@ def linear(x, w, bias=None, act: int = ACT_NONE, gated: bool = False, act_start:
             y = y + residual
         return y
     if not reduce:
-        return ref.linear(x, w, bias, act, gated, act_start, residual, out_dtype)
+        y = ref.linear(x, w, bias, act, gated, act_start, residual, out_dtype)
+        return y if out is None else out.copy_(y)
     y = ref.linear(x, w, None, ACT_NONE, False, 0, None, torch.float32)
     comm.all_reduce(y)
     if bias is not None:
@@ -312,18 +314,20 @@ def qknorm_kv_write(qkv, hq, hkv, dk, dv, q_w, k_w, eps, temp_coef, temp_every, 
 
 
 def attention_bias(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, dist_bias, gate=None, out_dtype=None, bias_over_scale=None,
-                   window=0, slopes=None, sinks=None):
+                   window=0, slopes=None, sinks=None, keep_first=0, softcap=0.0, diff=None, out=None):
     """Causal paged attention with separate key / value sizes, a per-head distance bias (a table, and / or a linear
     penalty ``slopes[h] * distance``), an optional sliding window, an output gate and an attention sink per head
     (``sinks`` [hq] 32-bit: exp(sinks[h]) joins every softmax denominator of head h).
-    ``bias_over_scale``: dist_bias / scale, kept by the caller for the tensor-core kernels (derived per call if absent)."""
+    ``bias_over_scale``: dist_bias / scale, kept by the caller for the tensor-core kernels (derived per call if absent).
+    ``keep_first``: first tokens that the window never hides; ``softcap``: cap * tanh(score / cap); ``diff`` = (lam, eps, factor): two
+    maps per head, combined as rms_div(a1 - lam * a2) * factor; ``out``: view that receives [T, hq * dv]."""
     if _cuda(q):
         from . import cuda_impl as cu
 
         return cu.attention_bias(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, dist_bias, gate, out_dtype, bias_over_scale,
-                                 window, slopes, sinks)
+                                 window, slopes, sinks, keep_first, softcap, diff, out)
     return ref.attention_bias(q, k_cache, v_cache, batch.block_tables, batch.seq_lens, batch.cu_q, hq, hkv, dk, dv, scale,
-                              dist_bias, gate, out_dtype, window, slopes, sinks)
+                              dist_bias, gate, out_dtype, window, slopes, sinks, keep_first, softcap, diff, out)
 
 
 def unary(x, op, out_dtype=None):
@@ -400,6 +404,24 @@ def sandwich_residual(resid, y, w_post, eps, w_next=None, history=None, index=0,
 def softcap(z, cap):
     """cap * tanh(z / cap) in place."""
     return _dispatch("softcap", z, z, cap)
+
+
+def residual_norm(resid, y, weight, bias, eps, kind, out_dtype=None):
+    """norm_residual over a 32-bit residual stream: (norm(resid + y) in ``out_dtype``, resid + y)."""
+    return _dispatch("residual_norm", resid, resid, y, weight, bias, eps, kind, out_dtype)
+
+
+def norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, interleaved, positions, slot_mapping, k_cache, v_cache,
+                       batch=None, out_dtype=None):
+    """Optional RMS norm with a weight per head (and map), rotation by a frequency table, keys and values to their pages; hkv = 0
+    prepares queries only.  ``batch`` lets the CUDA path lay the queries out for the attention kernel that will read them."""
+    if _cuda(qkv):
+        from . import cuda_impl as cu
+
+        return cu.norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, interleaved, positions, slot_mapping, k_cache,
+                                     v_cache, batch, out_dtype)
+    return ref.norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, interleaved, positions, slot_mapping, k_cache,
+                                  v_cache, out_dtype)
 
 
 def sample(logits, greedy, temperature, top_k, top_p, rng_state, vocab: Optional[int] = None, out=None):

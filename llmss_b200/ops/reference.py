@@ -612,16 +612,29 @@ def window_bias_table(slopes, window: int, scale: float):
 
 
 def attention_bias(q, k_cache, v_cache, block_tables, seq_lens, cu_q, hq: int, hkv: int, dk: int, dv: int, scale: float,
-                   dist_bias, gate=None, out_dtype=None, window: int = 0, slopes=None, sinks=None):
+                   dist_bias, gate=None, out_dtype=None, window: int = 0, slopes=None, sinks=None, keep_first: int = 0,
+                   softcap: float = 0.0, diff=None, out=None):
     """Causal softmax attention over the paged cache with key size dk, value size dv, grouped heads, an additive bias
     dist_bias[h, min(i - j, last)] per head and distance (or none), a linear penalty slopes[h] * (i - j) taken off the
     scores (or none), a sliding window (``window`` > 0: query i sees keys j with 0 <= i - j < window), an optional
     per-head output gate sigmoid(gate[t, h]), and an optional attention sink: ``sinks`` [hq] is a bare logit per head whose
     exponential is one more term of every softmax denominator of that head (nothing is added to the numerator, and the
-    score scale does not apply to it)."""
+    score scale does not apply to it).  ``keep_first``: with a window, the first ``keep_first`` tokens of the sequence stay
+    visible.  ``softcap`` > 0: the scaled score s becomes softcap * tanh(s / softcap) before anything is added to it.
+    ``diff`` = (lam, eps, factor): every head has two query / key maps of size dk over its one value (q [T, hq * 2 * dk], K pages
+    [.., 2 * dk], map 1 first); with a1, a2 the maps' outputs the head's output is rms_div(a1 - lam * a2) * factor.
+    ``out``: [T, hq * dv] view that receives the result."""
+    if diff is not None:
+        lam, eps, factor = diff
+        nb, _, bs, dk2 = k_cache.shape
+        halves = [attention_bias(q.reshape(-1, hq, 2, dk)[:, :, m].reshape(-1, hq * dk), k_cache[..., m * dk:(m + 1) * dk], v_cache,
+                                 block_tables, seq_lens, cu_q, hq, hkv, dk, dv, scale, dist_bias, gate, torch.float32, window, slopes,
+                                 sinks, keep_first, softcap).view(-1, hq, dv) for m in (0, 1)]
+        o = (_rms_div(halves[0] - lam * halves[1], eps) * factor).reshape(-1, hq * dv).to(out_dtype or q.dtype)
+        return o if out is None else out.copy_(o)
     T = q.shape[0]
     bs, g = k_cache.shape[2], hq // hkv
-    out = torch.zeros(T, hq, dv, dtype=torch.float32, device=q.device)
+    dst, out = out, torch.zeros(T, hq, dv, dtype=torch.float32, device=q.device)
     cu, lens = cu_q.tolist(), seq_lens.tolist()
     for i, L in enumerate(lens):
         q0, q1 = cu[i], cu[i + 1]
@@ -634,6 +647,8 @@ def attention_bias(q, k_cache, v_cache, block_tables, seq_lens, cu_q, hq: int, h
         v = v_cache[blocks].permute(1, 0, 2, 3).reshape(hkv, nb * bs, dv)[:, :L].float().repeat_interleave(g, dim=0)
         qi = q[q0:q1].float().view(ql, hq, dk).permute(1, 0, 2)
         s = torch.matmul(qi, k.transpose(1, 2)) * scale
+        if softcap > 0:
+            s = softcap * torch.tanh(s / softcap)
         qpos = torch.arange(L - ql, L, device=q.device)[:, None]
         kpos = torch.arange(L, device=q.device)[None, :]
         if dist_bias is not None:
@@ -643,7 +658,7 @@ def attention_bias(q, k_cache, v_cache, block_tables, seq_lens, cu_q, hq: int, h
             s = s - slopes.float()[:, None, None] * (qpos - kpos).float()[None]
         hidden = kpos > qpos
         if window > 0:
-            hidden = hidden | (qpos - kpos >= window)
+            hidden = hidden | ((qpos - kpos >= window) & (kpos >= keep_first))
         s = s.masked_fill(hidden, float("-inf"))
         if sinks is not None:
             p = torch.softmax(torch.cat([s, sinks.float().view(hq, 1, 1).expand(hq, ql, 1)], dim=-1), dim=-1)[..., :L]
@@ -652,7 +667,8 @@ def attention_bias(q, k_cache, v_cache, block_tables, seq_lens, cu_q, hq: int, h
         out[q0:q1] = torch.matmul(p, v).permute(1, 0, 2)
     if gate is not None:
         out = out * torch.sigmoid(gate.float())[:, :, None]
-    return out.reshape(T, hq * dv).to(out_dtype or q.dtype)
+    out = out.reshape(T, hq * dv).to(out_dtype or q.dtype)
+    return out if dst is None else dst.copy_(out)
 
 
 def unary(x, op: int, out_dtype=None):
@@ -796,7 +812,10 @@ def rotary_frequencies(dims: int, base: float, scaling=None):
     position interpolation); {"factor", "original", "fast", "slow"} blends per frequency (YaRN): with
     dim(t) = dims ln(original / (2 pi t)) / (2 ln base), lo = max(floor(dim(fast)), 0), hi = min(ceil(dim(slow)), dims - 1)
     and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1) the frequency is f_i / factor * ramp_i + f_i (1 - ramp_i) and
-    the magnitude 0.1 ln(factor) + 1.  The kernels take the table, so any other schedule is a different table."""
+    the magnitude 0.1 ln(factor) + 1; {"factor", "original", "low", "high"} goes by the wavelength l_i = 2 pi / f_i (Llama 3.1): f_i
+    stays below original / high, becomes f_i / factor above original / low, and is (1 - s) f_i / factor + s f_i with
+    s = (original / l_i - low) / (high - low) between the two.  The kernels take the table, so any other schedule is a
+    different table."""
     i = torch.arange(dims // 2, dtype=torch.float64)
     f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / dims)
     if not scaling:
@@ -804,6 +823,11 @@ def rotary_frequencies(dims: int, base: float, scaling=None):
     factor = float(scaling["factor"])
     if "original" not in scaling:
         return f / factor, 1.0
+    if "low" in scaling:
+        orig, low, high = float(scaling["original"]), float(scaling["low"]), float(scaling["high"])
+        turns = orig * f / (2.0 * math.pi)           # original / wavelength
+        mix = (turns - low) / (high - low) if high != low else torch.zeros_like(f)
+        return torch.where(turns > high, f, torch.where(turns < low, f / factor, (1.0 - mix) * f / factor + mix * f)), 1.0
     orig, fast, slow = float(scaling["original"]), float(scaling["fast"]), float(scaling["slow"])
 
     def at(t):
@@ -920,3 +944,39 @@ def sandwich_residual(resid, y, w_post, eps: float, w_next=None, history=None, i
 def softcap(z, cap: float):
     """cap * tanh(z / cap), in place on 32-bit logits."""
     return z.copy_(cap * torch.tanh(z.float() / cap))
+
+
+# ----------------------------------------------------------------------------- norms over a 32-bit residual, normed and rotated q / k
+def residual_norm(resid, y, weight, bias, eps: float, kind: int, out_dtype=None):
+    """norm_residual over a 32-bit residual stream: r = resid + y (y None: r = resid), h = LayerNorm or RMS norm of r.
+    Returns (h in ``out_dtype``, r 32-bit)."""
+    h, r = norm_residual(resid, y, weight, bias, eps, kind, out_dtype=torch.float32)
+    return h.to(out_dtype or torch.float32), r
+
+
+def norm_rope_kv_write(qkv, hq: int, hkv: int, dk: int, dv: int, maps: int, q_w, k_w, eps: float, freq, mag: float, interleaved: bool,
+                       positions, slot_mapping, k_cache, v_cache, out_dtype=None):
+    """Queries, keys and values of grouped-query attention from the fused 32-bit projection qkv [T, hq*maps*dk | hkv*maps*dk |
+    hkv*dv].  Every head has ``maps`` query / key vectors of size dk, side by side.  Each is divided by its root mean square and
+    multiplied by the weight q_w / k_w [dk] (None: no norm), then rotated by the frequency table; keys go to the K pages
+    [blocks, hkv, block_size, maps * dk], the values as they are to the V pages.  hkv = 0: queries only (a layer that attends
+    over another layer's pages).  Returns the queries [T, hq * maps * dk]."""
+    T = qkv.shape[0]
+
+    def prepare(x, w):
+        x = x.float()
+        if w is not None:
+            x = _rms_div(x, eps) * w.float()
+        return _rotate_by_table(x, positions, freq, mag, interleaved)
+
+    q = prepare(qkv[:, :hq * maps * dk].reshape(T, hq * maps, dk), q_w)
+    if hkv > 0:
+        lo = (hq + hkv) * maps * dk
+        k = prepare(qkv[:, hq * maps * dk:lo].reshape(T, hkv * maps, dk), k_w).reshape(T, hkv, maps * dk)
+        v = qkv[:, lo:lo + hkv * dv].reshape(T, hkv, dv)
+        bs = k_cache.shape[2]
+        valid = slot_mapping >= 0
+        slots = slot_mapping[valid].long()
+        k_cache[slots // bs, :, slots % bs, :] = k[valid].to(k_cache.dtype)
+        v_cache[slots // bs, :, slots % bs, :] = v[valid].to(v_cache.dtype)
+    return q.reshape(T, hq * maps * dk).to(out_dtype or k_cache.dtype)

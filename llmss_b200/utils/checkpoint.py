@@ -465,6 +465,86 @@ PRESETS.update({
 })
 
 
+def rofulorn_config(width: int, vocab: int, layers, embed_scale: float = 1.0, eps: float = 1e-6) -> dict:
+    """config.json of a Rofulorn model.  ``layers``: one dict per layer,
+    {"type": "attention", heads, kv_heads, dim, vdim, window, keep_first, diff, optionally softcap, kv_from} |
+    {"type": "attention_2", heads, kv_heads, dim, vdim, window}, each optionally with rot_dims, base, scaling {"factor", "low", "high",
+    "original"}, scale, and with "mlp": None | {"ff"}."""
+    out = []
+    for L in layers:
+        d = L["dim"]
+        rot = {"base": L.get("base", 10000.0), "dims": L.get("rot_dims", d)}
+        if L.get("scaling"):
+            rot["scaling"] = dict(L["scaling"])
+        m = {k: L[k] for k in ("heads", "kv_heads", "dim", "vdim")}
+        m.update(rot=rot, scale=L.get("scale", d ** -0.5), mask={"size": L["window"]})
+        if L["type"] == "attention":
+            m["mask"]["keep_first"] = L["keep_first"]
+            m["diff"] = L["diff"]
+            if L.get("softcap"):
+                m["softcap"] = L["softcap"]
+            if L.get("kv_from") is not None:
+                m["kv_from"] = L["kv_from"]
+        f = L.get("mlp")
+        out.append({"type": L["type"], "mixer": m, "mlp": None if f is None else {"kind": "dense", "ff": f["ff"]}})
+    return {"architecture": "Rofulorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "embedding": {"scale": embed_scale},
+            "layers": out}
+
+
+def _rofulorn_shapes(cfg: dict):
+    W, V = cfg["width"], cfg["vocab"]
+    yield "embed", (V, W), ("n", 0.0, 1.0 / cfg["embedding"]["scale"])
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}", L["mixer"]
+        q, d, dv, H, G = f"{p}.mix", m["dim"], m["vdim"], m["heads"], m["kv_heads"]
+        maps, own = (2 if "diff" in m else 1), m.get("kv_from") is None
+        yield f"{p}.norm1", (W,), "ln_w"
+        for s, n in (("q", H * maps * d),) + ((("k", G * maps * d), ("v", G * dv)) if own else ()):
+            yield f"{q}.{s}", (n, W), "fan"
+            if maps == 2:
+                yield f"{q}.{s}.b", (n,), ("n", 0.0, 0.1)
+        if maps == 2:
+            for s in ("q", "k") if own else ("q",):
+                yield f"{q}.{s}.norm", (d,), "ln_w"
+            for s in ("lq1", "lk1", "lq2", "lk2"):
+                yield f"{q}.{s}", (d,), ("n", 0.0, 0.1)
+            yield f"{q}.o.b", (W,), ("n", 0.0, 0.1)
+        yield f"{q}.o", (W, H * dv), "fan"
+        if L.get("mlp") is not None:
+            F = L["mlp"]["ff"]
+            yield f"{p}.mlp.gate", (F, W), "fan"
+            yield f"{p}.mlp.up", (F, W), "fan"
+            yield f"{p}.mlp.down", (W, F), "fan"
+    yield "final.norm", (W,), "ln_w"
+    yield "head", (V, W), "fan"
+
+
+def _rofulorn_preset(width, vocab, heads, ff, n_blocks, window=1024, kv_div=4):
+    """``n_blocks`` x (plain, differential, plain, differential on the pages of the block's second layer), each with a gated
+    feed-forward; head size 128 (plain) and 2 x 64 over values of 128 (differential)."""
+    G = max(1, heads // kv_div)
+    pln = dict(type="attention_2", heads=heads, kv_heads=G, dim=128, vdim=128, rot_dims=64, base=500000.0, window=window, mlp={"ff": ff})
+    dif = dict(type="attention", heads=heads, kv_heads=G, dim=64, vdim=128, rot_dims=32, window=2 * window, keep_first=8, diff=0.45,
+               softcap=30.0, scaling={"factor": 4.0, "low": 1.0, "high": 4.0, "original": 4096}, mlp={"ff": ff})
+    layers = []
+    for b in range(n_blocks):
+        layers += [dict(pln), dict(dif), dict(pln), dict(dif, kv_from=4 * b + 1)]
+    return rofulorn_config(width, vocab, layers, embed_scale=width ** 0.5)
+
+
+PRESETS.update({
+    "rofulorn-tiny": rofulorn_config(128, 320, [
+        dict(type="attention", heads=4, kv_heads=2, dim=24, vdim=40, rot_dims=16, window=20, keep_first=3, diff=0.4, softcap=20.0,
+             scaling={"factor": 4.0, "low": 1.0, "high": 4.0, "original": 64}, mlp={"ff": 192}),
+        dict(type="attention_2", heads=4, kv_heads=1, dim=32, vdim=24, rot_dims=24, window=33, mlp={"ff": 160}),
+        dict(type="attention", heads=6, kv_heads=2, dim=24, vdim=40, rot_dims=16, window=12, keep_first=5, diff=0.7, kv_from=0, mlp=None)],
+        embed_scale=8.0),
+    # sizes whose layers resemble a served model's (random weights), beside gptj-like-* of equal width and depth
+    "rofulorn-2k": _rofulorn_preset(2048, 32000, 16, 6144, 5),
+    "rofulorn-4k": _rofulorn_preset(4096, 32000, 32, 10240, 4),
+})
+
+
 def _shapes(cfg: dict) -> Iterator[Tuple[str, Tuple[int, ...], str]]:
     """(name, shape, kind) for every tensor of the family; kind in {w, b, ln_w, ln_b, emb} (and, for architectures whose
     activations must keep unit scale without trained weights: unit, fan, fan2, alpha, ls)."""
@@ -477,6 +557,8 @@ def _shapes(cfg: dict) -> Iterator[Tuple[str, Tuple[int, ...], str]]:
         yield from _botalorn_shapes(cfg)
     elif mt == "zenorax":
         yield from _zenorax_shapes(cfg)
+    elif mt == "rofulorn":
+        yield from _rofulorn_shapes(cfg)
     elif mt == "gptj":
         H, L, V = cfg["n_embd"], cfg["n_layer"], cfg["vocab_size"]
         F = cfg.get("n_inner") or 4 * H
