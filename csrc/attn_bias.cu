@@ -10,7 +10,10 @@
 //                     one pair: lane = key inside the tile for the scores, lane = output channel (mod 32) for P V.
 //                     Scores, softmax and accumulation are 32-bit with full-precision exponentials.
 //                     Optional: a linear penalty slopes[h] * (i - j) taken off the scores, and a sliding window (keys with
-//                     i - j >= window are hidden; the key loop starts at the first row's window).
+//                     i - j >= window are hidden; the key loop starts at the first row's window) that may keep the sequence's
+//                     first tokens, soft-capped scores cap * tanh(s / cap), and two query / key maps per head side by side in
+//                     the key row (the values are the head's; one output per map).
+//   diff_combine    : the two maps' outputs of a head -> rms_div(a1 - lam * a2) * factor.
 //   qkv_prepare     : the general form of qknorm_kv_write, one CTA per token: query / key norm per head or over the token's
 //                     whole projection, a factor per query head, values divided by their per-head root mean square, queries
 //                     only (no keys / values) for a layer that attends over another layer's pages.
@@ -133,12 +136,15 @@ struct AbArgs {
   int window;                             // > 0: only keys with i - j < window are visible
   const float* gate; int64_t ldg;         // [T][hq] logits, or null
   const float* sinks;                     // [hq] sink logits (one more term exp(sinks[h]) in every denominator), or null
-  void* out;                              // [T][hq * dv]
+  void* out; int64_t ldo;                 // [T][hq * dv], row stride ldo
   int hq, hkv, dk, dv, nh, rows, hsub;    // nh: query heads per CTA; rows: query rows per CTA; hsub: CTAs per kv head
   float scale;
+  int maps;                               // query heads h = head * maps + map read columns [map * dk, (map + 1) * dk) of the key row
+  int keep;                               // with a window: keys j < keep are visible whatever their distance
+  float cap;                              // > 0: scaled score s -> cap * tanh(s / cap), before bias and slopes
 };
 
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(NW * 32) attention_bias_kernel(AbArgs a) {
   extern __shared__ float sm[];
   const int b = blockIdx.z;
@@ -148,9 +154,9 @@ __global__ void __launch_bounds__(NW * 32) attention_bias_kernel(AbArgs a) {
   const int g = blockIdx.y / a.hsub, hs = blockIdx.y % a.hsub;
   const int gsz = a.hq / a.hkv;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int dk = a.dk, dv = a.dv, dkp = dk + 1;
+  const int dk = a.dk, dv = a.dv, dkr = a.dk * a.maps, dkp = dkr + 1;     // dkr: width of a key row
   float* qs = sm;                      // [NW][dk]
-  float* ks = qs + NW * dk;            // [TK][dk + 1]
+  float* ks = qs + NW * dk;            // [TK][dkr + 1]
   float* vs = ks + TK * dkp;           // [TK][dv]
   // this warp's (row, head)
   const int hl = warp % a.nh, rl = warp / a.nh;
@@ -173,14 +179,18 @@ __global__ void __launch_bounds__(NW * 32) attention_bias_kernel(AbArgs a) {
   const float* brow = a.bias != nullptr ? a.bias + (int64_t)(active ? h : 0) * a.n_dist : nullptr;
   const float slope = a.slopes != nullptr && active ? a.slopes[h] : 0.f;
   const int kbeg = a.window > 0 ? max(0, ctx + r0 - a.window + 1) : 0;      // first key any row of this CTA sees
-  const int klo = a.window > 0 ? qpos - a.window + 1 : 0;                   // first key this warp's row sees
-  for (int k0 = kbeg; k0 < kend; k0 += TK) {
-    const int nk = min(TK, kend - k0);
+  const int klo = a.window > 0 ? qpos - a.window + 1 : 0;                   // first key of this warp's row's window
+  const int kfirst = min(a.keep, kbeg);                                     // kept keys in front of the window: [0, kfirst)
+  const int kcol = a.maps > 1 ? (h % a.maps) * dk : 0;
+  int k1 = 0;                                                               // end of the tile = start of the next one
+  for (int k0 = kfirst > 0 ? 0 : kbeg; k0 < kend; k0 = (k1 >= kfirst && k1 < kbeg) ? kbeg : k1) {
+    const int nk = min(TK, (k0 < kfirst ? kfirst : kend) - k0);
+    k1 = k0 + nk;
     __syncthreads();
-    for (int idx = threadIdx.x; idx < nk * dk; idx += NW * 32) {
-      const int kk = idx / dk, c = idx % dk, pos = k0 + kk;
+    for (int idx = threadIdx.x; idx < nk * dkr; idx += NW * 32) {
+      const int kk = idx / dkr, c = idx % dkr, pos = k0 + kk;
       const int blk = a.block_tables[(int64_t)b * a.max_blocks + pos / a.bs];
-      ks[kk * dkp + c] = to_f32(kc[(((int64_t)blk * a.hkv + g) * a.bs + pos % a.bs) * dk + c]);
+      ks[kk * dkp + c] = to_f32(kc[(((int64_t)blk * a.hkv + g) * a.bs + pos % a.bs) * dkr + c]);
     }
     for (int idx = threadIdx.x; idx < nk * dv; idx += NW * 32) {
       const int kk = idx / dv, c = idx % dv, pos = k0 + kk;
@@ -188,15 +198,15 @@ __global__ void __launch_bounds__(NW * 32) attention_bias_kernel(AbArgs a) {
       vs[kk * dv + c] = to_f32(vc[(((int64_t)blk * a.hkv + g) * a.bs + pos % a.bs) * dv + c]);
     }
     __syncthreads();
-    if (!active || k0 > qpos || k0 + nk <= klo) continue;
+    if (!active || k0 > qpos || (k1 <= klo && k0 >= a.keep)) continue;
     const int kpos = k0 + lane;
     float sc = -INFINITY;
-    if (lane < nk && kpos <= qpos && kpos >= klo) {
+    if (lane < nk && kpos <= qpos && (kpos >= klo || kpos < a.keep)) {
       float d = 0.f;
-      const float* kr = ks + lane * dkp;
+      const float* kr = ks + lane * dkp + kcol;
       const float* qr = qs + warp * dk;
       for (int c = 0; c < dk; ++c) d = fmaf(qr[c], kr[c], d);
-      sc = d;
+      sc = a.cap > 0.f ? a.cap * tanhf(d / a.cap) : d;
       if (brow != nullptr) sc += brow[min(qpos - kpos, a.n_dist - 1)];
       sc -= slope * (float)(qpos - kpos);
     }
@@ -228,11 +238,37 @@ __global__ void __launch_bounds__(NW * 32) attention_bias_kernel(AbArgs a) {
     gsc = corr / (l * corr + expf(sk - mn));
   }
   if (a.gate != nullptr) gsc *= 1.f / (1.f + expf(-a.gate[(int64_t)(q0 + row) * a.ldg + h]));
-  T* og = reinterpret_cast<T*>(a.out) + (int64_t)(q0 + row) * a.hq * dv + (int64_t)h * dv;
+  TO* og = reinterpret_cast<TO*>(a.out) + (int64_t)(q0 + row) * a.ldo + (int64_t)h * dv;
 #pragma unroll
   for (int i = 0; i < MAXV; ++i) {
     const int c = lane + 32 * i;
-    if (c < dv) og[c] = from_f32<T>(acc[i] * gsc);
+    if (c < dv) og[c] = from_f32<TO>(acc[i] * gsc);
+  }
+}
+
+// One warp per (token, head): o = a1 - lam * a2 over the head's dv values, divided by its root mean square, times factor.
+// x [T][hq][2][dv] 32-bit.
+template <typename T>
+__global__ void __launch_bounds__(256) diff_combine_kernel(const float* __restrict__ x, int hq, int dv, float lam, float eps, float factor,
+                                                           T* __restrict__ out, int64_t ldo, int64_t units) {
+  const int64_t u = (int64_t)blockIdx.x * NW + (threadIdx.x >> 5);
+  if (u >= units) return;
+  const int lane = threadIdx.x & 31;
+  const float* a1 = x + u * 2 * dv;
+  const float* a2 = a1 + dv;
+  float v[MAXV], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int c = lane + 32 * i;
+    v[i] = c < dv ? fmaf(-lam, a2[c], a1[c]) : 0.f;
+    ss = fmaf(v[i], v[i], ss);
+  }
+  const float r = rsqrtf(warp_sum(ss) / (float)dv + eps) * factor;
+  T* o = out + (u / hq) * ldo + (u % hq) * dv;
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int c = lane + 32 * i;
+    if (c < dv) o[c] = from_f32<T>(v[i] * r);
   }
 }
 
@@ -285,7 +321,8 @@ static int attention_bias_launch(const void* q, int64_t ldq, const void* k_cache
                                  int max_blocks, int block_size, const int* seq_lens, const int* cu_q, const float* bias,
                                  int n_dist, const float* slopes, int window, const float* gate, int64_t ldg, void* out, int B,
                                  int max_q, int hq, int hkv, int dk, int dv, float scale, int dtype, cudaStream_t stream,
-                                 const float* sinks = nullptr) {
+                                 const float* sinks = nullptr, int maps = 1, int keep = 0, float cap = 0.f, int64_t ldo = 0,
+                                 int out_f32 = 0) {
   LLMSS_REQUIRE(hq > 0 && hkv > 0 && hq % hkv == 0, "attention_bias: %d query heads over %d key/value heads", hq, hkv);
   LLMSS_REQUIRE(dv <= 32 * MAXV, "attention_bias: value size %d (at most %d)", dv, 32 * MAXV);
   LLMSS_REQUIRE(bias == nullptr || n_dist > 0, "attention_bias: empty bias table");
@@ -295,23 +332,27 @@ static int attention_bias_launch(const void* q, int64_t ldq, const void* k_cache
   a.bs = block_size; a.seq_lens = seq_lens; a.cu_q = cu_q; a.bias = bias; a.n_dist = n_dist; a.slopes = slopes; a.window = window; a.gate = gate; a.ldg = ldg; a.out = out;
   a.sinks = sinks;
   a.hq = hq; a.hkv = hkv; a.dk = dk; a.dv = dv; a.scale = scale;
+  a.maps = maps; a.keep = keep; a.cap = cap; a.ldo = ldo > 0 ? ldo : (int64_t)hq * dv;
   const int gsz = hq / hkv;
   a.nh = gsz < NW ? gsz : NW;
   a.rows = NW / a.nh;
   a.hsub = (gsz + NW - 1) / NW;
-  const size_t smem = sizeof(float) * ((size_t)NW * dk + (size_t)TK * (dk + 1) + (size_t)TK * dv);
+  const size_t smem = sizeof(float) * ((size_t)NW * dk + (size_t)TK * (dk * maps + 1) + (size_t)TK * dv);
   LLMSS_REQUIRE(smem <= 200 * 1024, "attention_bias: key size %d / value size %d exceed shared memory", dk, dv);
   const dim3 grid((max_q + a.rows - 1) / a.rows, hkv * a.hsub, B);
   LLMSS_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "attention_bias: grid too large");
-#define LLMSS_AB(TT)                                                                \
+#define LLMSS_AB(TT, TO)                                                                \
   do {                                                                              \
     static PerDeviceSmem gsm;                                                       \
-    LLMSS_CHECK_CUDA(gsm.ensure(attention_bias_kernel<TT>, (int)smem));             \
-    attention_bias_kernel<TT><<<grid, NW * 32, smem, stream>>>(a);                  \
+    auto kern = attention_bias_kernel<TT, TO>;                                      \
+    LLMSS_CHECK_CUDA(gsm.ensure(kern, (int)smem));                                  \
+    kern<<<grid, NW * 32, smem, stream>>>(a);                                       \
   } while (0)
-  if (dtype == LLMSS_F16) LLMSS_AB(__half);
-  else if (dtype == LLMSS_BF16) LLMSS_AB(__nv_bfloat16);
-  else if (dtype == LLMSS_F32) LLMSS_AB(float);
+  if (dtype == LLMSS_F16 && out_f32) LLMSS_AB(__half, float);
+  else if (dtype == LLMSS_F16) LLMSS_AB(__half, __half);
+  else if (dtype == LLMSS_BF16 && out_f32) LLMSS_AB(__nv_bfloat16, float);
+  else if (dtype == LLMSS_BF16) LLMSS_AB(__nv_bfloat16, __nv_bfloat16);
+  else if (dtype == LLMSS_F32) LLMSS_AB(float, float);
   else LLMSS_REQUIRE(false, "bad dtype %d", dtype);
 #undef LLMSS_AB
   LLMSS_CHECK_CUDA(cudaGetLastError());
@@ -345,4 +386,29 @@ LLMSS_API int llmss_attention_sink(const void* q, int64_t ldq, const void* k_cac
   LLMSS_REQUIRE(window >= 0, "attention_sink: window %d", window);
   return attention_bias_launch(q, ldq, k_cache, v_cache, block_tables, max_blocks, block_size, seq_lens, cu_q, bias, n_dist, slopes,
                                window, gate, ldg, out, B, max_q, hq, hkv, dk, dv, scale, dtype, stream, sinks);
+}
+
+// the same with everything at once: a window that keeps the sequence's first `keep_first` tokens, soft-capped scores (cap > 0) and
+// `maps` query / key vectors per head (hq counts heads x maps: query head h is map h % maps; key rows are maps * dk wide, the
+// key / value head of query head h is h / (hq / hkv)).  out [T][hq * dv] with row stride ldo, 32-bit if out_f32.
+LLMSS_API int llmss_attention_span(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
+                                   int max_blocks, int block_size, const int* seq_lens, const int* cu_q, int window, int keep_first,
+                                   float cap, int maps, void* out, int64_t ldo, int out_f32, int B, int max_q, int hq, int hkv, int dk,
+                                   int dv, float scale, int dtype, cudaStream_t stream) {
+  LLMSS_REQUIRE(window >= 0 && keep_first >= 0 && cap >= 0.f && maps >= 1 && hkv > 0 && (hq / hkv) % maps == 0,
+                "attention_span: window %d, keep_first %d, cap %f, %d maps, %d query heads", window, keep_first, cap, maps, hq);
+  return attention_bias_launch(q, ldq, k_cache, v_cache, block_tables, max_blocks, block_size, seq_lens, cu_q, nullptr, 0, nullptr, window,
+                               nullptr, 0, out, B, max_q, hq, hkv, dk, dv, scale, dtype, stream, nullptr, maps, keep_first, cap, ldo, out_f32);
+}
+
+// x [T][hq][2][dv] 32-bit -> out [T][hq * dv] (row stride ldo): rms_div(x1 - lam * x2) * factor per head
+LLMSS_API int llmss_diff_combine(const float* x, int T_, int hq, int dv, float lam, float eps, float factor, void* out, int64_t ldo,
+                                 int dtype, cudaStream_t stream) {
+  LLMSS_REQUIRE(hq > 0 && dv > 0 && dv <= 32 * MAXV, "diff_combine: value size %d (at most %d)", dv, 32 * MAXV);
+  if (T_ <= 0) return 0;
+  const int64_t units = (int64_t)T_ * hq;
+  LLMSS_BY_DTYPE(dtype, (diff_combine_kernel<T><<<(unsigned)((units + NW - 1) / NW), NW * 32, 0, stream>>>(x, hq, dv, lam, eps, factor,
+                                                                                                          (T*)out, ldo, units)));
+  LLMSS_CHECK_CUDA(cudaGetLastError());
+  return 0;
 }

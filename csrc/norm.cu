@@ -101,7 +101,135 @@ __global__ void __launch_bounds__(kThreads) norm_residual_kernel(
   }
 }
 
+// ------------------------------------------------------------------------------------------------ 32-bit residual stream
+// r = resid + y (y null: r = resid) ; h = LayerNorm / RMS norm of r times weight (+ bias), stored as TO.  One CTA per row, the
+// row in registers (VEC = 4: 16-byte accesses; longer rows are read back from `out_r`), two-pass variance, 32-bit throughout.
+struct RnArgs {
+  const float* resid; int64_t ldr;
+  const float* y; int64_t ldy;
+  const float* w; const float* bias;
+  float* out_r; void* out_h;         // [M, W] contiguous; out_r null: r is not stored (y null)
+  int W; float eps; int kind;
+};
+constexpr int kRnRegs = 4;
+
+template <int VEC> __device__ __forceinline__ void rn_load(const float* p, float (&v)[VEC]) {
+  if constexpr (VEC == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+  } else v[0] = p[0];
+}
+
+template <typename TO, int VEC>
+__global__ void __launch_bounds__(kThreads) residual_norm_kernel(RnArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[kThreads / 32];
+  const int64_t t = blockIdx.x;
+  const int W = a.W;
+  constexpr int STEP = kThreads * VEC;
+  float keep[kRnRegs][VEC];
+  float sum = 0.f;
+  const bool rms = a.kind == LLMSS_NORM_RMS;
+  auto fetch = [&](int c, float (&v)[VEC]) {
+    rn_load<VEC>(a.resid + t * a.ldr + c, v);
+    if (a.y != nullptr) {
+      float u[VEC];
+      rn_load<VEC>(a.y + t * a.ldy + c, u);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[e] += u[e];
+    }
+    if (a.out_r != nullptr) {
+      float* o = a.out_r + t * (int64_t)W + c;
+      if constexpr (VEC == 4) *reinterpret_cast<float4*>(o) = make_float4(v[0], v[1], v[2], v[3]);
+      else o[0] = v[0];
+    }
+  };
+  const float* again = a.out_r != nullptr ? a.out_r + t * (int64_t)W : a.resid + t * a.ldr;   // this thread's own columns of r
+#pragma unroll
+  for (int i = 0; i < kRnRegs; ++i) {
+    const int c = threadIdx.x * VEC + i * STEP;
+    if (c < W) {
+      fetch(c, keep[i]);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) sum += rms ? keep[i][e] * keep[i][e] : keep[i][e];
+    }
+  }
+  for (int c = threadIdx.x * VEC + kRnRegs * STEP; c < W; c += STEP) {
+    float v[VEC];
+    fetch(c, v);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) sum += rms ? v[e] * v[e] : v[e];
+  }
+  float mean = 0.f, rstd;
+  if (rms) {
+    rstd = rsqrtf(block_sum(sum, red) / (float)W + a.eps);
+  } else {
+    mean = block_sum(sum, red) / (float)W;
+    float sq = 0.f;
+#pragma unroll
+    for (int i = 0; i < kRnRegs; ++i) {
+      const int c = threadIdx.x * VEC + i * STEP;
+      if (c < W) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) { const float d = keep[i][e] - mean; sq = fmaf(d, d, sq); }
+      }
+    }
+    for (int c = threadIdx.x * VEC + kRnRegs * STEP; c < W; c += STEP) {
+      float v[VEC];
+      rn_load<VEC>(again + c, v);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) { const float d = v[e] - mean; sq = fmaf(d, d, sq); }
+    }
+    rstd = rsqrtf(block_sum(sq, red) / (float)W + a.eps);
+  }
+  auto emit = [&](int c, const float (&v)[VEC]) {
+    float wv[VEC], bv[VEC];
+    rn_load<VEC>(a.w + c, wv);
+    if (a.bias != nullptr) rn_load<VEC>(a.bias + c, bv);
+    TO* ho = reinterpret_cast<TO*>(a.out_h) + t * (int64_t)W + c;
+    struct alignas(VEC * sizeof(TO)) Pack { TO v[VEC]; };
+    Pack o;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      const float h = (v[e] - mean) * rstd * wv[e];
+      o.v[e] = from_f32<TO>(a.bias != nullptr ? h + bv[e] : h);
+    }
+    *reinterpret_cast<Pack*>(ho) = o;
+  };
+#pragma unroll
+  for (int i = 0; i < kRnRegs; ++i) {
+    const int c = threadIdx.x * VEC + i * STEP;
+    if (c < W) emit(c, keep[i]);
+  }
+  for (int c = threadIdx.x * VEC + kRnRegs * STEP; c < W; c += STEP) {
+    float v[VEC];
+    rn_load<VEC>(again + c, v);
+    emit(c, v);
+  }
+}
+
+template <typename TO>
+int residual_norm_launch(const RnArgs& a, int M, bool vec, cudaStream_t stream) {
+  if (vec) LLMSS_CHECK_CUDA(launch_pdl(residual_norm_kernel<TO, 4>, dim3(M), dim3(kThreads), 0, stream, a));
+  else LLMSS_CHECK_CUDA(launch_pdl(residual_norm_kernel<TO, 1>, dim3(M), dim3(kThreads), 0, stream, a));
+  return 0;
+}
+
 }  // namespace
+
+// The counterpart of llmss_norm_residual over a 32-bit residual stream: resid [M, W] (row stride ldr), y [M, W] or null, weight /
+// bias 32-bit (bias may be null), out_r [M, W] contiguous (null with y null), out_h [M, W] contiguous in out_dtype.
+LLMSS_API int llmss_residual_norm(const float* resid, int64_t ldr, const float* y, int64_t ldy, const float* weight, const float* bias,
+                                  float* out_r, void* out_h, int M, int W, float eps, int kind, int out_dtype, cudaStream_t stream) {
+  LLMSS_REQUIRE(W > 0 && weight != nullptr && out_h != nullptr && (y == nullptr || out_r != nullptr), "residual_norm: bad arguments");
+  LLMSS_REQUIRE(kind == LLMSS_NORM_LAYER || kind == LLMSS_NORM_RMS, "residual_norm: norm kind %d", kind);
+  if (M <= 0) return 0;
+  RnArgs a{resid, ldr, y, ldy, weight, bias, out_r, out_h, W, eps, kind};
+  const bool vec = W % 4 == 0 && ldr % 4 == 0 && ldy % 4 == 0 &&
+                   ((((uintptr_t)resid) | ((uintptr_t)y) | ((uintptr_t)weight) | ((uintptr_t)bias) | ((uintptr_t)out_r) | ((uintptr_t)out_h)) & 15) == 0;
+  LLMSS_BY_DTYPE(out_dtype, return (residual_norm_launch<T>(a, M, vec, stream)));
+}
 
 LLMSS_API int llmss_norm_residual(const void* x, const void* x2, const void* residual_in, void* residual_out,
                                   const void* weight, const void* bias, void* out, int M, int H, int64_t ldx,

@@ -3,6 +3,9 @@
 //   rope_norm_kv_write : grouped-query attention whose values are the projected keys.  q and k are rotated (pairs (2i, 2i+1) or
 //                        (i, i + n)), optionally every head is divided by its root mean square, the prepared keys go to the K
 //                        pages, the raw key projection to the V pages, the queries out in the compute type.
+//   norm_rope_kv_write : q, k, v of grouped-query attention: optional RMS norm of every query / key vector with a weight shared by
+//                        the heads, rotation, keys and values to their pages; one or several query / key vectors ("maps") per
+//                        head side by side; queries only for a layer that attends over another layer's pages.
 //   latent_rope_prep   : latent attention with a rotated key part, first stage: RMS norm of the query latent (-> GEMM operand),
 //                        RMS norm of the key / value latent and rotation of the shared key part (-> one cache row), sigmoid of
 //                        the gate columns.
@@ -120,6 +123,123 @@ __global__ void __launch_bounds__(256) rope_norm_kv_write_kernel(const float* __
       for (int c = lane; c < d; c += 32) {
         k_cache[base + c] = from_f32<T>(rotated(x, c, n, interleaved, cs, sn) * rstd);
         v_cache[base + c] = from_f32<T>(x[c]);
+      }
+    }
+  }
+}
+
+// norm_rope_kv_write: grid T, block 256, a warp per vector of the token's row (hq * maps queries, hkv * maps keys, hkv values).
+// VEC: interleaved pairs and sizes that are multiples of four -- a lane holds its 4-column groups in registers from the 16-byte
+// load to the store; otherwise the row is re-read element by element.
+struct NrArgs {
+  const float* qkv; int64_t ld;
+  int hq, hkv, dk, dv, maps;
+  const float* q_w; const float* k_w;     // [dk] or null: no norm
+  float eps;
+  const double* freq; int n; float mag; int interleaved;
+  const int* positions; const int* slots;
+  void* k_cache; void* v_cache; int bs;
+  void* q_out;
+  int pad;                                // queries as [hq * maps][maps * dk], zero outside the map's own columns
+};
+constexpr int kNrVec = 4;                 // 4-column groups per lane: dk <= 512 in the vector form
+
+template <typename T> struct alignas(4 * sizeof(T)) Quad { T v[4]; };
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
+  __shared__ float cs[kMaxPairs], sn[kMaxPairs];
+  const int64_t t = blockIdx.x;
+  token_angles(a.freq, a.n, a.positions[t], a.mag, cs, sn);
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int dk = a.dk, dv = a.dv, nq = a.hq * a.maps, nk = a.hkv * a.maps, row = a.maps * dk;
+  const int slot = a.hkv > 0 ? a.slots[t] : -1;
+  const int64_t page = slot >= 0 ? (int64_t)(slot / a.bs) * a.hkv * a.bs + slot % a.bs : 0;    // row index of key/value head 0
+  T* kc = reinterpret_cast<T*>(a.k_cache);
+  T* vc = reinterpret_cast<T*>(a.v_cache);
+  for (int u = warp; u < nq + nk + a.hkv; u += 8) {
+    if (u >= nq && slot < 0) continue;
+    if (u >= nq + nk) {                                          // a value vector: as projected
+      const int g = u - nq - nk;
+      const float* x = a.qkv + t * a.ld + (int64_t)(nq + nk) * dk + (int64_t)g * dv;
+      T* dst = vc + (page + (int64_t)g * a.bs) * dv;
+      if constexpr (VEC) {
+        for (int c = lane * 4; c < dv; c += 128) {
+          const float4 v = *reinterpret_cast<const float4*>(x + c);
+          Quad<T> o{from_f32<T>(v.x), from_f32<T>(v.y), from_f32<T>(v.z), from_f32<T>(v.w)};
+          *reinterpret_cast<Quad<T>*>(dst + c) = o;
+        }
+      } else {
+        for (int c = lane; c < dv; c += 32) dst[c] = from_f32<T>(x[c]);
+      }
+      continue;
+    }
+    const bool is_q = u < nq;
+    const int hm = is_q ? u : u - nq, m = hm % a.maps;
+    const float* x = a.qkv + t * a.ld + (int64_t)u * dk;
+    const float* w = is_q ? a.q_w : a.k_w;
+    T* dst;
+    if (is_q) dst = reinterpret_cast<T*>(a.q_out) + (a.pad ? (t * nq + hm) * (int64_t)row + m * dk : (t * nq + hm) * (int64_t)dk);
+    else dst = kc + (page + (int64_t)(hm / a.maps) * a.bs) * row + m * dk;
+    if constexpr (VEC) {
+      float v[kNrVec][4];
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < kNrVec; ++i) {
+        const int c = lane * 4 + i * 128;
+        if (c < dk) {
+          const float4 f = *reinterpret_cast<const float4*>(x + c);
+          v[i][0] = f.x; v[i][1] = f.y; v[i][2] = f.z; v[i][3] = f.w;
+          ss = fmaf(f.x, f.x, fmaf(f.y, f.y, fmaf(f.z, f.z, fmaf(f.w, f.w, ss))));
+        }
+      }
+      const float rstd = w != nullptr ? rsqrtf(warp_sum(ss) / (float)dk + a.eps) : 1.f;
+#pragma unroll
+      for (int i = 0; i < kNrVec; ++i) {
+        const int c = lane * 4 + i * 128;
+        if (c >= dk) continue;
+        if (w != nullptr) {
+          const float4 wv = *reinterpret_cast<const float4*>(w + c);
+          v[i][0] *= rstd * wv.x; v[i][1] *= rstd * wv.y; v[i][2] *= rstd * wv.z; v[i][3] *= rstd * wv.w;
+        }
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const int pr = (c + e) >> 1;
+          if (pr < a.n) {
+            const float p = v[i][e], q = v[i][e + 1], cc = cs[pr], ssn = sn[pr];
+            v[i][e] = fmaf(p, cc, -q * ssn);
+            v[i][e + 1] = fmaf(q, cc, p * ssn);
+          }
+        }
+        Quad<T> o{from_f32<T>(v[i][0]), from_f32<T>(v[i][1]), from_f32<T>(v[i][2]), from_f32<T>(v[i][3])};
+        *reinterpret_cast<Quad<T>*>(dst + c) = o;
+        if (is_q && a.pad) {                                     // zeros where the other maps' columns are
+          const Quad<T> z{from_f32<T>(0.f), from_f32<T>(0.f), from_f32<T>(0.f), from_f32<T>(0.f)};
+          for (int o2 = 0; o2 < a.maps; ++o2)
+            if (o2 != m) *reinterpret_cast<Quad<T>*>(dst + (o2 - m) * dk + c) = z;
+        }
+      }
+    } else {
+      float rstd = 1.f;
+      if (w != nullptr) {
+        float ss = 0.f;
+        for (int c = lane; c < dk; c += 32) ss = fmaf(x[c], x[c], ss);
+        rstd = rsqrtf(warp_sum(ss) / (float)dk + a.eps);
+      }
+      auto normed = [&](int c) { return w != nullptr ? x[c] * (rstd * w[c]) : x[c]; };
+      for (int c = lane; c < dk; c += 32) {
+        float r = normed(c);
+        if (c < 2 * a.n) {
+          const bool second = a.interleaved ? (c & 1) : c >= a.n;
+          const int pr = a.interleaved ? c >> 1 : (second ? c - a.n : c);
+          const float o = normed(a.interleaved ? (c ^ 1) : (second ? c - a.n : c + a.n));
+          r = second ? fmaf(r, cs[pr], o * sn[pr]) : fmaf(r, cs[pr], -o * sn[pr]);
+        }
+        dst[c] = from_f32<T>(r);
+        if (is_q && a.pad)
+          for (int o2 = 0; o2 < a.maps; ++o2)
+            if (o2 != m) dst[(o2 - m) * dk + c] = from_f32<T>(0.f);
       }
     }
   }
@@ -356,6 +476,31 @@ LLMSS_API int llmss_rope_norm_kv_write(const float* qk, int64_t ld, int hq, int 
     LLMSS_BY_DTYPE(dtype, (rope_norm_kv_write_kernel<T, false><<<T_, 256, 0, stream>>>(
                               qk, ld, hq, hkv, d, freq, n_pairs, mag, interleaved, unit_norm, eps, positions, slots, (T*)k_cache,
                               (T*)v_cache, block_size, (T*)q_out)));
+  }
+  LLMSS_CHECK_CUDA(cudaGetLastError());
+  return 0;
+}
+
+// qkv [T][hq*maps*dk | hkv*maps*dk | hkv*dv] 32-bit; q_w / k_w [dk] 32-bit or null (no norm); K pages [blocks][hkv][block_size][maps *
+// dk], V pages [blocks][hkv][block_size][dv]; q_out [T][hq*maps][dk], or [T][hq*maps][maps*dk] with zeros outside the map's own
+// columns (pad = 1).  hkv = 0: queries only.
+LLMSS_API int llmss_norm_rope_kv_write(const float* qkv, int64_t ld, int hq, int hkv, int dk, int dv, int maps, const float* q_w,
+                                       const float* k_w, float eps, const double* freq, int n_pairs, float mag, int interleaved,
+                                       const int* positions, const int* slots, void* k_cache, void* v_cache, int block_size, void* q_out,
+                                       int pad, int T_, int dtype, cudaStream_t stream) {
+  LLMSS_REQUIRE(hq > 0 && hkv >= 0 && dk > 0 && maps >= 1 && (hkv == 0 || dv > 0), "norm_rope_kv_write: bad sizes");
+  LLMSS_REQUIRE(hkv == 0 || (k_cache != nullptr && v_cache != nullptr && slots != nullptr && block_size > 0), "norm_rope_kv_write: keys without pages");
+  LLMSS_REQUIRE(n_pairs >= 0 && n_pairs <= kMaxPairs && 2 * n_pairs <= dk, "norm_rope_kv_write: %d rotated pairs for head size %d (at most %d)",
+                n_pairs, dk, kMaxPairs);
+  if (T_ <= 0) return 0;
+  NrArgs a{qkv, ld, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, n_pairs, mag, interleaved, positions, slots, k_cache, v_cache,
+           block_size, q_out, pad};
+  const bool vec = interleaved && dk % 4 == 0 && dk <= 128 * kNrVec && (hkv == 0 || dv % 4 == 0) && ld % 4 == 0 &&
+                   ((((uintptr_t)qkv) | ((uintptr_t)q_w) | ((uintptr_t)k_w) | ((uintptr_t)k_cache) | ((uintptr_t)v_cache) | ((uintptr_t)q_out)) & 15) == 0;
+  if (vec) {
+    LLMSS_BY_DTYPE(dtype, (norm_rope_kv_write_kernel<T, true><<<T_, 256, 0, stream>>>(a)));
+  } else {
+    LLMSS_BY_DTYPE(dtype, (norm_rope_kv_write_kernel<T, false><<<T_, 256, 0, stream>>>(a)));
   }
   LLMSS_CHECK_CUDA(cudaGetLastError());
   return 0;

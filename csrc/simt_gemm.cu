@@ -25,6 +25,7 @@ struct BgArgs {
   int64_t ssh, ssn;                      // (1, 0): one factor per (token, head); (N, 1): one per output element
   void* out; int64_t ldo, soh;
   int M, N, K, H, act, act_start;
+  int gated;                             // rows of w interleave (gate, up): out column n / 2 = act(gate) * up
 };
 
 __device__ __forceinline__ float act_sq(float x, int act) {
@@ -83,6 +84,17 @@ __global__ void __launch_bounds__(NT) bgemm_kernel(BgArgs a) {
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + ty * 4 + i;
     if (m >= a.M) continue;
+    if (a.gated) {     // a thread's four columns are two (gate, up) pairs
+#pragma unroll
+      for (int j = 0; j < 4; j += 2) {
+        const int n = n0 + tx * 4 + j;
+        if (n + 1 >= a.N) continue;
+        float gv = acc[i][j], uv = acc[i][j + 1];
+        if (bias != nullptr) { gv += to_f32(bias[n]); uv += to_f32(bias[n + 1]); }
+        out[(int64_t)m * a.ldo + (n >> 1)] = from_f32<TO>(act_sq(gv, a.act) * uv);
+      }
+      continue;
+    }
     const float* rsp = a.row_scale != nullptr ? a.row_scale + (int64_t)m * a.lds + (int64_t)h * a.ssh : nullptr;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
@@ -251,7 +263,7 @@ LLMSS_API int llmss_bgemm_simt_ex(const void* x, int64_t ldx, int64_t sxh, const
   LLMSS_REQUIRE(M >= 0 && N > 0 && K > 0 && H > 0 && H <= 65535, "bgemm_simt: bad shape M=%d N=%d K=%d H=%d", M, N, K, H);
   LLMSS_REQUIRE((M + BM - 1) / BM <= 65535, "bgemm_simt: M=%d too large", M);
   if (M == 0) return 0;
-  BgArgs a{x, ldx, sxh, w, swh, swk, swn, bias, row_scale, lds, ssh, ssn, out, ldo, soh, M, N, K, H, act, act_start};
+  BgArgs a{x, ldx, sxh, w, swh, swk, swn, bias, row_scale, lds, ssh, ssn, out, ldo, soh, M, N, K, H, act, act_start, 0};
   // 16-bit operands without bias / activation (the per-head products) take the tensor-core form; the 32-bit accumulators
   // are the same, so both forms agree to rounding of the summation order
   const bool mma_ok = dtype != LLMSS_F32 && bias == nullptr && act == LLMSS_ACT_NONE && (M + 127) / 128 <= 65535;
@@ -269,4 +281,17 @@ LLMSS_API int llmss_bgemm_simt(const void* x, int64_t ldx, int64_t sxh, const vo
                                int dtype, int out_f32, cudaStream_t stream) {
   return llmss_bgemm_simt_ex(x, ldx, sxh, w, swh, swk, swn, bias, row_scale, lds, 1, 0, out, ldo, soh, M, N, K, H, act, act_start,
                              dtype, out_f32, stream);
+}
+
+// Gated linear layer on the CUDA cores: out[t, n] = act(x_t . w_(2n)) * (x_t . w_(2n+1)), w [2 * n_out, K] with interleaved
+// (gate, up) rows (row stride ldw); true 32-bit, or 16-bit operands off the 16-byte rules of the tensor-core GEMM.
+LLMSS_API int llmss_gated_simt(const void* x, int64_t ldx, const void* w, int64_t ldw, const void* bias, void* out, int64_t ldo, int M,
+                               int n_out, int K, int act, int dtype, cudaStream_t stream) {
+  LLMSS_REQUIRE(M >= 0 && n_out > 0 && K > 0 && (M + BM - 1) / BM <= 65535, "gated_simt: bad shape M=%d N=%d K=%d", M, n_out, K);
+  if (M == 0) return 0;
+  BgArgs a{x, ldx, 0, w, 0, 1, ldw, bias, nullptr, 0, 1, 0, out, ldo, 0, M, 2 * n_out, K, 1, act, 0, 1};
+  if (dtype == LLMSS_F32) return launch_bg<float>(a, 1, stream);
+  if (dtype == LLMSS_BF16) return launch_bg<__nv_bfloat16>(a, 0, stream);
+  if (dtype == LLMSS_F16) return launch_bg<__half>(a, 0, stream);
+  LLMSS_REQUIRE(false, "gated_simt: bad dtype %d", dtype);
 }

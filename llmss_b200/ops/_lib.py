@@ -176,6 +176,17 @@ _SIGS = {
     "llmss_softcap": (c_int, [c_void_p, c_int64, c_int, c_int, c_float, c_void_p]),
     "llmss_sandwich_residual": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                         c_void_p, c_int, c_int, c_float, c_int, c_void_p]),
+    "llmss_residual_norm": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float,
+                                    c_int, c_int, c_void_p]),
+    "llmss_norm_rope_kv_write": (c_int, [c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p,
+                                         c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
+                                         c_int, c_void_p]),
+    "llmss_attention_span": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
+                                     c_float, c_int, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
+                                     c_int, c_void_p]),
+    "llmss_diff_combine": (c_int, [c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p, c_int64, c_int, c_void_p]),
+    "llmss_gated_simt": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int,
+                                 c_void_p]),
 }
 _OPTIONAL = {
     "llmss_attn_decode_tc_sink": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int64,

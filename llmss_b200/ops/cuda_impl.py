@@ -114,11 +114,18 @@ def _needs_simt(x, w, K, ldx, ldw) -> bool:
 def linear_simt(x, w, bias=None, act: int = ACT_NONE, gated: bool = False, act_start: int = 0, residual=None,
                 out_dtype=None, out=None):
     """The same linear layer on the CUDA cores (csrc/simt_gemm.cu): true 32-bit, or shapes the tcgen05 kernel refuses."""
-    if gated:
-        raise NotImplementedError("the CUDA-core GEMM has no gated epilogue")
     lib = _lib.load()
     M, K, ldx = _rows2d(x)
     N, _, ldw = _rows2d(w)
+    if gated:
+        assert residual is None and out_dtype in (None, x.dtype) and N % 2 == 0
+        if out is None:
+            out = torch.empty(M, N // 2, dtype=x.dtype, device=x.device)
+        assert out.dtype == x.dtype and out.stride(1) == 1
+        rc = lib.llmss_gated_simt(_ptr(x), ldx, _ptr(w), ldw, _ptr(bias), _ptr(out), out.stride(0), M, N // 2, K, act, _DT[x.dtype], _stream())
+        _lib.check(rc, "llmss_gated_simt")
+        _count()
+        return out
     f32 = x.dtype == torch.float32 or out_dtype == torch.float32
     if out is None:
         out = torch.empty(M, N, dtype=torch.float32 if f32 else x.dtype, device=x.device)
@@ -880,7 +887,11 @@ from .reference import window_bias_table  # noqa: E402  (the window and slopes a
 
 
 def attention_bias(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, dist_bias, gate=None, out_dtype=None, bias_over_scale=None,
-                   window=0, slopes=None, sinks=None):
+                   window=0, slopes=None, sinks=None, keep_first=0, softcap=0.0, diff=None, dst=None):
+    if keep_first or softcap or diff is not None or dst is not None or (window and slopes is None and dist_bias is None):
+        assert dist_bias is None and slopes is None and gate is None and sinks is None, \
+            "attention: kept first tokens, soft cap and two-map heads have no bias, slopes, gate or sink beside them"
+        return attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window or 0, keep_first, softcap, diff, out_dtype, dst)
     lib = _lib.load()
     T = q.shape[0]
     dt = q.dtype
@@ -962,6 +973,70 @@ def attention_bias(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, dist_bias
     _lib.check(rc, "llmss_attention_bias")
     _count()
     return out
+
+
+# --------------------------------------------------------------------------- windows with kept first tokens, soft cap, two maps per head
+def attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window=0, keep_first=0, softcap=0.0, diff=None, out_dtype=None,
+                   out=None):
+    """attention_bias without additive terms; see ops.reference.attention_bias for window, keep_first, softcap and diff."""
+    lib = _lib.load()
+    T, dt, bs = q.shape[0], q.dtype, k_cache.shape[2]
+    maps = 1 if diff is None else 2
+    assert k_cache.dtype == dt and (out_dtype or dt) == dt and q.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert k_cache.shape[1] == hkv and k_cache.shape[3] == maps * dk and v_cache.shape[3] == dv
+    if out is None:
+        out = torch.empty(T, hq * dv, dtype=dt, device=q.device)
+    assert out.dtype == dt and out.shape == (T, hq * dv) and out.stride(1) == 1
+    # the generic kernel: any sizes, true 32-bit; the two maps' outputs stay in 32-bit until they are combined
+    o = torch.empty(T, hq * maps * dv, dtype=torch.float32, device=q.device) if maps == 2 else out
+    rc = lib.llmss_attention_span(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables), batch.block_tables.shape[1],
+                                  bs, _ptr(batch.seq_lens), _ptr(batch.cu_q), int(window), int(keep_first), float(softcap), maps, _ptr(o),
+                                  o.stride(0), 1 if maps == 2 else 0, batch.num_seqs, max(1, batch.max_q), hq * maps, hkv, dk, dv,
+                                  float(scale), _DT[dt], _stream())
+    _lib.check(rc, "llmss_attention_span")
+    _count()
+    if maps == 2:
+        lam, eps, factor = diff
+        _lib.check(lib.llmss_diff_combine(_ptr(o), T, hq, dv, float(lam), float(eps), float(factor), _ptr(out), out.stride(0), _DT[dt],
+                                          _stream()), "llmss_diff_combine")
+        _count()
+    return out
+
+
+def residual_norm(resid, y, weight, bias, eps, kind, out_dtype=None):
+    lib = _lib.load()
+    T, W, ldr = _f32rows(resid)
+    dt = out_dtype or torch.float32
+    assert weight.dtype == torch.float32 and weight.numel() == W and (bias is None or bias.dtype == torch.float32)
+    ldy = 0
+    if y is not None:
+        _, Wy, ldy = _f32rows(y)
+        assert Wy == W
+    h = torch.empty(T, W, dtype=dt, device=resid.device)
+    r = torch.empty(T, W, dtype=torch.float32, device=resid.device) if y is not None else resid
+    rc = lib.llmss_residual_norm(_ptr(resid), ldr, _ptr(y), ldy, _ptr(weight), _ptr(bias), _ptr(r) if y is not None else None, _ptr(h), T, W,
+                                 float(eps), int(kind), _DT[dt], _stream())
+    _lib.check(rc, "llmss_residual_norm")
+    _count()
+    return h, r
+
+
+def norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, interleaved, positions, slot_mapping, k_cache, v_cache,
+                       batch=None, out_dtype=None):
+    lib = _lib.load()
+    T, _, ld = _f32rows(qkv)
+    dt = out_dtype or k_cache.dtype
+    assert k_cache.dtype == dt and v_cache.dtype == dt and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert k_cache.shape[3] == maps * dk and (hkv == 0 or (k_cache.shape[1] == hkv and v_cache.shape[3] == dv))
+    assert all(w is None or (w.dtype == torch.float32 and w.numel() == dk) for w in (q_w, k_w))
+    pad = 0
+    q = torch.empty(T, hq * maps * dk, dtype=dt, device=qkv.device)
+    rc = lib.llmss_norm_rope_kv_write(_ptr(qkv), ld, hq, hkv, dk, dv, maps, _ptr(q_w), _ptr(k_w), float(eps),
+                                      _ptr(_freq_dev(freq, qkv.device)), freq.numel(), float(mag), 1 if interleaved else 0, _ptr(positions),
+                                      _ptr(slot_mapping), _ptr(k_cache), _ptr(v_cache), k_cache.shape[2], _ptr(q), pad, T, _DT[dt], _stream())
+    _lib.check(rc, "llmss_norm_rope_kv_write")
+    _count()
+    return q
 
 
 # --------------------------------------------------------------------------- rotation by a table, sandwich norms
