@@ -17,6 +17,11 @@
 // partially filled page still enter the PV MMA multiplied by P = 0, so cache pages must hold finite values
 // (0 * NaN = NaN).  The engine zero-initialises the pool and pages only ever hold real K/V, so this holds.
 //
+// Span form (llmss_attn_decode_span): a sliding window -- only the key tiles it reaches, and those of the sequence's kept first
+// tokens, are walked --, soft-capped scores, key and value sizes that are any multiple of 8 (the tile is the next of 64 / 128 /
+// 256, columns beyond the size arrive as TMA's zero fill), and two query / key maps per head: the key row holds both maps, the
+// query rows come zero-padded to that width, so a group's 2 G rows share one read of K and V; the combine pass subtracts.
+//
 // Replaces SURVEY.md G8 (`baddbmm` + TorchScript softmax + `bmm` on a replicated KV tensor,
 // gpt_bigcode_modeling.py:170-246) and G7 for grouped models.
 #include "common.cuh"
@@ -63,10 +68,18 @@ struct DArgs {
   int dtype;
   const float* sinks;  // optional attention sink per q head: 2^(sinks[h] log2 e) joins the denominator (here when an item
                        // covers its whole sequence, else in the combine pass)
+  int dk, dv;          // key row / value size (<= the tile's D)
+  int k_ops, v_ops;    // TMA ops per page: 1, or one per 64-column chunk where the size is no multiple of 64
+  int k_tx, v_tx;      // bytes per key tile
+  int window, keep;    // span form: window 0: none; keys < keep are never hidden
+  float cap_in, cap_log2;   // soft cap: cap_in = scale / cap (0: none), cap_log2 = cap * log2 e
+  int partials;        // 1: write partials even when an item covers its whole sequence (the combine pass has more to do)
 };
 
 struct Item {
-  int b, kvh, split, L, t_begin, t_end, n_tiles;
+  int b, kvh, L, n_tiles;
+  int v_begin;          // first tile of this unit in the walk: tiles 0 .. n_first - 1, then t_first .. (see key_tile)
+  int t_first, n_first;
   int direct;   // this unit covers the whole sequence: write the normalised output, no partial
   int part;     // partial slot within the (sequence, head) row
   int pstride;  // slots per (sequence, head)
@@ -81,20 +94,26 @@ __device__ __forceinline__ int balanced_quota(int total_tiles, int grid) {
   return (total_tiles + active - 1) / active > 1 ? (total_tiles + active - 1) / active : 1;
 }
 
+__device__ __forceinline__ int key_tile(const Item& r, int j) {
+  const int v = r.v_begin + j;
+  return v < r.n_first ? v : v - r.n_first + r.t_first;
+}
+
 __device__ __forceinline__ Item decode_item(const DArgs& a, int it) {
   Item r;
-  r.split = it % a.num_splits;
+  const int split = it % a.num_splits;
   const int t = it / a.num_splits;
   r.kvh = t % a.hkv;
   r.b = t / a.hkv;
   r.L = a.seq_lens[r.b];
-  int chunk = (r.L + a.num_splits - 1) / a.num_splits;
-  chunk = (chunk + a.bn - 1) / a.bn * a.bn;  // whole key tiles per split
-  r.t_begin = r.split * chunk;
-  r.t_end = min(r.L, r.t_begin + chunk);
-  r.n_tiles = r.t_end > r.t_begin ? (r.t_end - r.t_begin + a.bn - 1) / a.bn : 0;
-  r.direct = a.num_splits == 1;
-  r.part = r.split;
+  r.t_first = a.window > 0 ? max(0, r.L - a.window) / a.bn : 0;
+  r.n_first = min((a.keep + a.bn - 1) / a.bn, r.t_first);
+  const int total = r.L > 0 ? (r.L + a.bn - 1) / a.bn - r.t_first + r.n_first : 0;
+  const int chunk = (total + a.num_splits - 1) / a.num_splits;  // whole key tiles per split
+  r.v_begin = split * chunk;
+  r.n_tiles = max(0, min(total - r.v_begin, chunk));
+  r.direct = a.num_splits == 1 && a.partials == 0;
+  r.part = split;
   r.pstride = a.num_splits;
   return r;
 }
@@ -145,10 +164,9 @@ struct Sched {
     const int take = (n - j) < (t_stop - t) ? (n - j) : (t_stop - t);
     r.b = b;
     r.kvh = kvh;
-    r.split = 0;
     r.L = a.seq_lens[b];
-    r.t_begin = j * a.bn;
-    r.t_end = r.L < (j + take) * a.bn ? r.L : (j + take) * a.bn;
+    r.v_begin = j;
+    r.t_first = r.n_first = 0;
     r.n_tiles = take;
     r.direct = take == n;
     r.part = (int)blockIdx.x - (t - j) / quota;  // CTAs that share this item are consecutive
@@ -208,15 +226,6 @@ __device__ __forceinline__ uint32_t pack2(float a, float b) {
   }
 }
 
-
-__device__ __forceinline__ void tma_load_3d(void* smem_dst, const void* map, uint64_t* bar, int c0, int c1, int c2,
-                                            uint64_t policy) {
-  asm volatile(
-      "cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes.L2::cache_hint"
-      " [%0], [%1, {%3, %4, %5}], [%2], %6;" ::"r"(smem_u32(smem_dst)),
-      "l"(map), "r"(smem_u32(bar)), "r"(c0), "r"(c1), "r"(c2), "l"(policy)
-      : "memory");
-}
 
 __device__ __forceinline__ uint64_t umma_desc_k_sw128_sbo(uint32_t smem_addr, uint32_t sbo_bytes) {
   uint64_t d = 0;
@@ -332,11 +341,11 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
       const int qb = n & 1;
       mbar_wait(&bar_qempty[qb], ((n >> 1) & 1) ^ 1, 40);
       if (elect_one()) {
-        mbar_arrive_expect_tx(&bar_qfull[qb], (uint32_t)(a.q_copies * a.q_box_rows * D * 2));
+        mbar_arrive_expect_tx(&bar_qfull[qb], (uint32_t)(a.q_copies * a.q_box_rows * ((a.dk + 63) / 64) * 128));
         for (int cc = 0; cc < a.q_copies; ++cc)
 #pragma unroll
           for (int c = 0; c < DSUB; ++c)
-            tma_load_3d(sQ + qb * q_bytes + c * q_chunk + cc * (a.q_box_rows * 128), &tmap_q, &bar_qfull[qb], c * 64,
+            if (c * 64 < a.dk) tma_load_3d(sQ + qb * q_bytes + c * q_chunk + cc * (a.q_box_rows * 128), &tmap_q, &bar_qfull[qb], c * 64,
                         I.kvh * G, I.b, pol_q);
       }
       // Block-table entries are fetched 32 pages at a time (one coalesced load per warp, the next group
@@ -344,10 +353,9 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
       const int* bt = a.block_tables + (int64_t)I.b * a.max_blocks;
       const int bs = a.block_size;
       const int last_page = (I.L - 1) / bs;
-      const int page_begin = I.t_begin / bs;
       const int tiles_per_group = 32 / pages;
       auto load_rows = [&](int group) {
-        const int pg = page_begin + group * 32 + lane;
+        const int pg = key_tile(I, group * tiles_per_group + lane / pages) * pages + lane % pages;
         // pages past the end of the sequence are masked later: fetch the reserved block 0 instead
         const int blk = (pg <= last_page) ? __ldg(bt + pg) : 0;
         return (blk * a.hkv + I.kvh) * bs;
@@ -360,20 +368,22 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
           if (j + tiles_per_group < I.n_tiles) nxt = load_rows(j / tiles_per_group + 1);
         }
         mbar_wait(&bar_kempty[stage], phase ^ 1, 50);
-        if (elect_one()) mbar_arrive_expect_tx(&bar_kfull[stage], KV_BYTES);
+        if (elect_one()) mbar_arrive_expect_tx(&bar_kfull[stage], (uint32_t)a.k_tx);
         __syncwarp();
         for (int p = 0; p < pages; ++p) {
           const int row = __shfl_sync(0xffffffffu, cur, tg * pages + p);
           if (elect_one())
-            tma_load_3d(sK + stage * KV_BYTES + p * (bs * D * 2), &tmap_k, &bar_kfull[stage], 0, row, 0, pol_kv);
+            for (int c = 0; c < a.k_ops; ++c)
+              tma_load_3d(sK + stage * KV_BYTES + p * (bs * D * 2) + c * (bs * 128), &tmap_k, &bar_kfull[stage], c * 64, row, 0, pol_kv);
         }
         mbar_wait(&bar_vempty[stage], phase ^ 1, 51);
-        if (elect_one()) mbar_arrive_expect_tx(&bar_vfull[stage], KV_BYTES);
+        if (elect_one()) mbar_arrive_expect_tx(&bar_vfull[stage], (uint32_t)a.v_tx);
         __syncwarp();
         for (int p = 0; p < pages; ++p) {
           const int row = __shfl_sync(0xffffffffu, cur, tg * pages + p);
           if (elect_one())
-            tma_load_3d(sV + stage * KV_BYTES + p * (bs * D * 2), &tmap_v, &bar_vfull[stage], 0, row, 0, pol_kv);
+            for (int c = 0; c < a.v_ops; ++c)
+              tma_load_3d(sV + stage * KV_BYTES + p * (bs * D * 2) + c * (bs * 128), &tmap_v, &bar_vfull[stage], c * 64, row, 0, pol_kv);
         }
         if (++stage == S) { stage = 0; phase ^= 1; }
       }
@@ -413,7 +423,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
             for (int c = 0; c < DSUB; ++c)
 #pragma unroll
               for (int k = 0; k < 4; ++k)
-                umma_f16_ss_ws(tS + (g & 1) * 16, umma_desc_k_sw128_sbo(q_addr + c * q_chunk + k * 32, a.q_sbo),
+                if (c * 64 + k * 16 < a.dk) umma_f16_ss_ws(tS + (g & 1) * 16, umma_desc_k_sw128_sbo(q_addr + c * q_chunk + k * 32, a.q_sbo),
                                umma_desc_k_sw128(k_addr + c * chunk_bytes + k * 32), idesc_ws, (c | k) ? 1u : 0u);
             umma_commit(&bar_s[g & 1]);
             umma_commit(&bar_kempty[kst]);
@@ -425,7 +435,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
             for (int c = 0; c < DSUB; ++c)
 #pragma unroll
               for (int k = 0; k < 4; ++k)
-                umma_f16_ss(tS + (g & 1) * BN + p * bs, umma_desc_k_sw128_sbo(q_addr + c * q_chunk + k * 32, a.q_sbo),
+                if (c * 64 + k * 16 < a.dk) umma_f16_ss(tS + (g & 1) * BN + p * bs, umma_desc_k_sw128_sbo(q_addr + c * q_chunk + k * 32, a.q_sbo),
                             umma_desc_k_sw128(k_addr + p * page_bytes + c * chunk_bytes + k * 32), idesc_s,
                             (c | k) ? 1u : 0u);
           umma_commit(&bar_s[g & 1]);
@@ -491,6 +501,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
     const int n_threads = n_live_warps * 32;
     const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
     uint32_t g = 0;
+    const float scale_log2 = a.cap_in > 0.f ? a.cap_log2 : a.scale_log2;
     Sched sch(a);
     Item I;
     while (sch.next(I)) {
@@ -499,8 +510,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
       if (I.n_tiles == 0) {  // empty split (or empty sequence): neutral partial / zero output
         if (live && owner) {
           if (I.direct) {
-            T* orow = reinterpret_cast<T*>(a.out) + (int64_t)I.b * a.ldo + (int64_t)head * D;
-            for (int c = 0; c < D; c += 8) *reinterpret_cast<uint4*>(orow + c) = make_uint4(0, 0, 0, 0);
+            T* orow = reinterpret_cast<T*>(a.out) + (int64_t)I.b * a.ldo + (int64_t)head * a.dv;
+            for (int c = 0; c < a.dv; c += 8) *reinterpret_cast<uint4*>(orow + c) = make_uint4(0, 0, 0, 0);
           } else {
             for (int c = 0; c < D; c += 4) *reinterpret_cast<float4*>(a.part_o + pidx * D + c) = make_float4(0, 0, 0, 0);
             a.part_ml[pidx * 2] = -INFINITY;
@@ -513,7 +524,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
       for (int j = 0; j < I.n_tiles; ++j, ++g) {
         mbar_wait(&bar_s[g & 1], (g >> 1) & 1, 70);
         tcgen05_fence_after();
-        const int kbase = I.t_begin + j * BN + c0;
+        const int kbase = key_tile(I, j) * BN + c0;
         float sc[CW];
         if constexpr (CW == 16) {
           uint32_t r[16];
@@ -535,10 +546,17 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
         tcgen05_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(&bar_sfree[g & 1]);  // S(g) is in registers: the buffer can take QK(g+2)
-        if (kbase + CW > I.t_end) {
+        if (a.cap_in > 0.f) softcap_scores<CW>(sc, a.cap_in);
+        if (kbase + CW > I.L) {
 #pragma unroll
           for (int i = 0; i < CW; ++i)
-            if (kbase + i >= I.t_end) sc[i] = -INFINITY;
+            if (kbase + i >= I.L) sc[i] = -INFINITY;
+        }
+        if (a.window > 0 && kbase < I.L - a.window && kbase + CW > a.keep) {   // the window starts inside or behind these keys
+          const int lo = I.L - a.window - kbase, kp = a.keep - kbase;
+#pragma unroll
+          for (int i = 0; i < CW; ++i)
+            if (i < lo && i >= kp) sc[i] = -INFINITY;
         }
         if (a.bias != nullptr && live) {
           const float* bt = a.bias + (int64_t)head * a.n_dist;
@@ -558,7 +576,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
         }
         // Lazy rescale: keep the old running max unless the tile exceeds it by more than 2^8, so the
         // accumulator is rarely touched and softmax(g+1) does not wait for PV(g).
-        const float m_tile_s = m_tile * a.scale_log2;
+        const float m_tile_s = m_tile * scale_log2;
         const bool grow = (j == 0) || (m_tile_s > m_run + 8.0f);
         const float m_new = grow ? fmaxf(m_run, m_tile_s) : m_run;
         float alpha = (j == 0 || !grow) ? 1.0f : ex2_approx(m_run - m_new);
@@ -573,8 +591,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
           uint32_t pk[4];
 #pragma unroll
           for (int i = 0; i < 8; i += 2) {
-            const float p0 = ex2_approx(fmaf(sc[c * 8 + i], a.scale_log2, neg_m));
-            const float p1 = ex2_approx(fmaf(sc[c * 8 + i + 1], a.scale_log2, neg_m));
+            const float p0 = ex2_approx(fmaf(sc[c * 8 + i], scale_log2, neg_m));
+            const float p1 = ex2_approx(fmaf(sc[c * 8 + i + 1], scale_log2, neg_m));
             l_tile += p0 + p1;
             pk[i >> 1] = pack2<T>(p0, p1);
           }
@@ -629,9 +647,10 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
         tmem_ld_wait();
         if (!live) continue;
         if (I.direct) {
-          T* orow = reinterpret_cast<T*>(a.out) + (int64_t)I.b * a.ldo + (int64_t)head * D + e_base;
+          T* orow = reinterpret_cast<T*>(a.out) + (int64_t)I.b * a.ldo + (int64_t)head * a.dv + e_base;
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
+            if (e_base + c * 32 + q * 8 >= a.dv) break;
             float f8[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) f8[i] = __uint_as_float(r[q * 8 + i]) * inv_l;
@@ -703,6 +722,50 @@ __global__ void attn_decode_tc_balanced_combine_kernel(const float* __restrict__
       at += part_o[(base + s) * D + c] * sc;
     }
     orow[c] = from_f32<T>(lt > 0.f ? at / (lt + sink_l) : 0.f);
+  }
+}
+
+// Span form: merges the splits of every query head; maps = 2: heads 2h and 2h + 1 are a head's maps and the result is
+// rms_div(a1 - lam * a2) * factor over the head's dv values.  Partials have row stride D.  grid (heads, B), 128 threads.
+template <typename T>
+__global__ void __launch_bounds__(128) attn_decode_span_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                                                                       T* __restrict__ out, int64_t ldo, int hq, int maps, int D, int dv,
+                                                                       int num_splits, float lam, float eps, float factor) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[4];
+  const int head = blockIdx.x, b = blockIdx.y;
+  float o[2] = {0.f, 0.f};                     // columns threadIdx.x and threadIdx.x + 128
+  for (int m = 0; m < maps; ++m) {
+    const int64_t base = ((int64_t)b * hq + head * maps + m) * num_splits;
+    float mn = -INFINITY;
+    for (int s = 0; s < num_splits; ++s) mn = fmaxf(mn, part_ml[(base + s) * 2]);
+    float lt = 0.f, at[2] = {0.f, 0.f};
+    for (int s = 0; s < num_splits; ++s) {
+      const float ms = part_ml[(base + s) * 2];
+      const float sc = (ms == -INFINITY) ? 0.f : exp2f(ms - mn);
+      lt += part_ml[(base + s) * 2 + 1] * sc;
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int c = threadIdx.x + i * 128;
+        if (c < dv) at[i] += part_o[(base + s) * D + c] * sc;
+      }
+    }
+    const float w = lt > 0.f ? (m == 0 ? 1.f : -lam) / lt : 0.f;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) o[i] = fmaf(at[i], w, o[i]);
+  }
+  float r = 1.f;
+  if (maps == 2) {
+    const float ss = warp_sum(o[0] * o[0] + o[1] * o[1]);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    r = rsqrtf((red[0] + red[1] + red[2] + red[3]) / (float)dv + eps) * factor;
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int c = threadIdx.x + i * 128;
+    if (c < dv) out[(int64_t)b * ldo + (int64_t)head * dv + c] = from_f32<T>(o[i] * r);
   }
 }
 
@@ -809,16 +872,23 @@ LLMSS_API int llmss_attn_decode_tc_supported(int hq, int hkv, int d, int block_s
 // Tensor-core (tcgen05) paged decode attention: the q heads of a KV group are MMA rows.  Same contract
 // as llmss_attn_decode; `scratch` holds the split-KV partials.  Requires block_size in {16, 32, 64}, head_dim in
 // {64, 128, 256}, hq / hkv <= 128.
+struct SpanArgs {
+  int dk, dv, maps;      // key row and value size; query / key maps per head (hq counts heads x maps)
+  int window, keep;
+  float cap, lam, eps, factor;
+};
+
 static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
                           int max_blocks, const int* seq_lens, void* out, int64_t ldo, float* scratch, int B, int hq, int hkv, int d,
                           int block_size, int num_blocks, float scale, int num_splits, int dtype, const float* bias, int n_dist,
-                          cudaStream_t stream, const float* sinks = nullptr) {
+                          cudaStream_t stream, const float* sinks = nullptr, const SpanArgs* span = nullptr) {
   LLMSS_REQUIRE(dtype == LLMSS_F16 || dtype == LLMSS_BF16, "attn_decode_tc: dtype must be f16/bf16");
   LLMSS_REQUIRE(d == 64 || d == 128 || d == 256, "attn_decode_tc: head_dim=%d unsupported", d);
   LLMSS_REQUIRE(hq > 0 && hkv > 0, "attn_decode_tc: head counts must be positive (hq=%d hkv=%d)", hq, hkv);
   LLMSS_REQUIRE(hq % hkv == 0 && hq / hkv <= 128, "attn_decode_tc: bad head grouping hq=%d hkv=%d", hq, hkv);
   LLMSS_REQUIRE(block_size == 16 || block_size == 32 || block_size == 64, "attn_decode_tc: block_size must be 16/32/64");
-  LLMSS_REQUIRE(num_splits >= 0 && (num_splits == 1 || scratch != nullptr), "attn_decode_tc: scratch required for splits");
+  LLMSS_REQUIRE(num_splits >= 0 && ((num_splits == 1 && (span == nullptr || span->maps == 1)) || scratch != nullptr),
+                "attn_decode_tc: scratch required for splits");
   const int balanced = num_splits == 0 ? 1 : 0;  // flat partition of all key tiles over the SMs
   const int max_parts = balanced_max_parts(max_blocks, block_size, tile_keys(d));
   LLMSS_REQUIRE(ldq % 8 == 0 && ldo % 8 == 0 && ((uintptr_t)q % 16) == 0, "attn_decode_tc: q must be 16-byte aligned");
@@ -835,12 +905,13 @@ static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const
   int smem = 0;
   const int stages = plan_stages(q_alloc_rows, d, &smem);
   LLMSS_REQUIRE(stages >= 2, "attn_decode_tc: shared memory too small for hq/hkv=%d d=%d", G, d);
+  const int dk = span != nullptr ? span->dk : d, dv = span != nullptr ? span->dv : d;
   const CUtensorMapDataType dt = dtype == LLMSS_BF16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
   CUtensorMap tq, tk, tv;
   {
     // q viewed as [B][hq][d]: box = [1][q_box_rows][64]
-    cuuint64_t dims[3] = {(cuuint64_t)d, (cuuint64_t)hq, (cuuint64_t)B};
-    cuuint64_t strides[2] = {(cuuint64_t)d * 2, (cuuint64_t)ldq * 2};
+    cuuint64_t dims[3] = {(cuuint64_t)dk, (cuuint64_t)hq, (cuuint64_t)B};
+    cuuint64_t strides[2] = {(cuuint64_t)dk * 2, (cuuint64_t)ldq * 2};
     cuuint32_t box[3] = {64, (cuuint32_t)q_box_rows, 1};
     cuuint32_t estr[3] = {1, 1, 1};
     CUresult r = enc(&tq, dt, 3, const_cast<void*>(q), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
@@ -850,10 +921,14 @@ static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const
   for (int which = 0; which < 2; ++which) {
     // cache viewed as [d/64 chunks][num_blocks * hkv * block_size rows][64]: one box = one page of one head,
     // landing in shared memory chunk-major ([chunk][block_size rows][128 B]), which is what the MMA
-    // descriptors of a page expect -- a single TMA op per page whatever the head size.
-    cuuint64_t dims[3] = {64, (cuuint64_t)num_blocks * hkv * block_size, (cuuint64_t)(d / 64)};
-    cuuint64_t strides[2] = {(cuuint64_t)d * 2, 128};
-    cuuint32_t box[3] = {64, (cuuint32_t)block_size, (cuuint32_t)(d / 64)};
+    // descriptors of a page expect -- a single TMA op per page whatever the head size.  A size that is no multiple of 64 goes
+    // chunk by chunk instead, so that the columns beyond it are out of the map's range and read as zeros.
+    const int w = which == 0 ? dk : dv;
+    const bool whole = w % 64 == 0;
+    const cuuint64_t rows = (cuuint64_t)num_blocks * hkv * block_size;
+    cuuint64_t dims[3] = {(cuuint64_t)(whole ? 64 : w), rows, (cuuint64_t)(whole ? w / 64 : 1)};
+    cuuint64_t strides[2] = {(cuuint64_t)w * 2, whole ? 128 : rows * w * 2};
+    cuuint32_t box[3] = {64, (cuuint32_t)block_size, (cuuint32_t)(whole ? w / 64 : 1)};
     cuuint32_t estr[3] = {1, 1, 1};
     CUresult r = enc(which == 0 ? &tk : &tv, dt, 3, const_cast<void*>(which == 0 ? k_cache : v_cache), dims, strides, box,
                      estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
@@ -893,6 +968,19 @@ static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const
   a.bias = bias;
   a.n_dist = n_dist;
   a.sinks = sinks;
+  a.dk = dk;
+  a.dv = dv;
+  a.k_ops = dk % 64 == 0 ? 1 : (dk + 63) / 64;
+  a.v_ops = dv % 64 == 0 ? 1 : (dv + 63) / 64;
+  a.k_tx = (dk + 63) / 64 * 128 * tile_keys(d);
+  a.v_tx = (dv + 63) / 64 * 128 * tile_keys(d);
+  if (span != nullptr) {
+    a.window = span->window < (1 << 30) ? span->window : 0;
+    a.keep = span->keep < (1 << 30) ? span->keep : (1 << 30);
+    a.cap_in = span->cap > 0.f ? scale / span->cap : 0.f;
+    a.cap_log2 = span->cap * 1.4426950408889634f;
+    a.partials = span->maps > 1 ? 1 : 0;
+  }
   int rc = 0;
 #define LLMSS_DT(T_, D_)                                                         \
   do {                                                                           \
@@ -910,7 +998,18 @@ static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const
     else LLMSS_DT(__nv_bfloat16, 256);
   }
 #undef LLMSS_DT
-  if (rc != 0 || num_splits == 1) return rc;
+  if (rc != 0 || (num_splits == 1 && a.partials == 0)) return rc;
+  if (span != nullptr) {
+    const dim3 cgrid(hq / span->maps, B);
+    if (dtype == LLMSS_F16)
+      LLMSS_CHECK_CUDA(launch_pdl(attn_decode_span_combine_kernel<__half>, cgrid, dim3(128), 0, stream, (const float*)a.part_o, (const float*)a.part_ml,
+                                  (__half*)out, ldo, hq, span->maps, d, dv, num_splits, span->lam, span->eps, span->factor));
+    else
+      LLMSS_CHECK_CUDA(launch_pdl(attn_decode_span_combine_kernel<__nv_bfloat16>, cgrid, dim3(128), 0, stream, (const float*)a.part_o,
+                                  (const float*)a.part_ml, (__nv_bfloat16*)out, ldo, hq, span->maps, d, dv, num_splits, span->lam, span->eps,
+                                  span->factor));
+    return 0;
+  }
   if (balanced) {
     const dim3 cgrid(hq, B);
     const int threads = d < 128 ? d : 128;
@@ -957,4 +1056,23 @@ LLMSS_API int llmss_attn_decode_tc_sink(const void* q, int64_t ldq, const void* 
   LLMSS_REQUIRE(scale > 0.f && (bias_over_scale == nullptr || n_dist > 0), "attn_decode_tc_sink: needs a positive scale");
   return decode_tc_impl(q, ldq, k_cache, v_cache, block_tables, max_blocks, seq_lens, out, ldo, scratch, B, hq, hkv, d, block_size,
                         num_blocks, scale, num_splits, dtype, bias_over_scale, n_dist, stream, sinks);
+}
+
+// Span form (one query token per sequence): see the head of the file.  q [B][hq * maps][maps * dk] -- for maps = 2 every row zero
+// outside its own map's columns --, K pages [num_blocks][hkv][block_size][maps * dk], V pages [..][dv], out [B][hq * dv] (row
+// stride ldo).  scratch: llmss_attn_decode_scratch_floats(B, hq * maps, D, num_splits) floats, D = 64 / 128 / 256 the smallest
+// that holds maps * dk and dv; needed for num_splits > 1 or maps = 2.  num_splits >= 1.
+LLMSS_API int llmss_attn_decode_span(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
+                                     int max_blocks, const int* seq_lens, void* out, int64_t ldo, float* scratch, int B, int hq, int hkv,
+                                     int dk, int dv, int maps, int block_size, int num_blocks, float scale, int window, int keep_first,
+                                     float cap, float lam, float eps, float factor, int num_splits, int dtype, cudaStream_t stream) {
+  LLMSS_REQUIRE(maps == 1 || maps == 2, "attn_decode_span: %d maps", maps);
+  LLMSS_REQUIRE(dk > 0 && dv > 0 && dk % 8 == 0 && dv % 8 == 0 && maps * dk <= 256 && dv <= 256,
+                "attn_decode_span: key size %d x %d / value size %d unsupported", maps, dk, dv);
+  LLMSS_REQUIRE(scale > 0.f && window >= 0 && keep_first >= 0 && cap >= 0.f && num_splits >= 1, "attn_decode_span: bad scale, window, cap or splits");
+  LLMSS_REQUIRE((((uintptr_t)out | (uintptr_t)k_cache | (uintptr_t)v_cache) % 16) == 0, "attn_decode_span: out / pages must be 16-byte aligned");
+  const int w = maps * dk > dv ? maps * dk : dv, d = w <= 64 ? 64 : (w <= 128 ? 128 : 256);
+  const SpanArgs sp{maps * dk, dv, maps, window, keep_first, cap, lam, eps, factor};
+  return decode_tc_impl(q, ldq, k_cache, v_cache, block_tables, max_blocks, seq_lens, out, ldo, scratch, B, hq * maps, hkv, d, block_size,
+                        num_blocks, scale, num_splits, dtype, nullptr, 0, stream, nullptr, &sp);
 }

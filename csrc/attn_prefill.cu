@@ -19,6 +19,15 @@
 //   q, k, v are column ranges of the packed QKV activation (row stride ld*), so the kernel reads
 //   the GEMM output in place; `out` may alias q (the fused GPT-J block writes the context over q).
 //   GQA/MQA: kv head = q head / (hq / hkv).
+//
+// Span form (MAPS = 1 / 2, over the paged cache): a sliding window whose hidden key tiles are skipped and that may keep the
+// sequence's first tokens (their tiles come first in the walk), soft-capped scores, and any key / value size that is a
+// multiple of 8 (the tile is the next of 64 / 128 / 256; TMA fills the columns beyond the size with zeros).  MAPS = 2 is
+// differential attention: a head has two query / key vectors over one value and the key row holds both side by side.  A CTA
+// takes 64 queries; rows 0-63 of its query tile are map 1 and rows 64-127 map 2, each zero outside its own half of the key
+// row (again TMA's fill: the box starts at a shifted column), so ONE MMA per tile forms the scores of both maps from one
+// read of K and V.  The epilogue hands the second map's rows over through shared memory, subtracts, divides by the root mean
+// square over the head and stores the 16-bit result: the two maps' outputs never leave the SM.
 #include "common.cuh"
 
 #include <cuda.h>
@@ -87,6 +96,11 @@ struct PArgs {
   int64_t ldg;
   // and an attention sink per head: 2^(sinks[h] * log2 e) joins every denominator of head h (a bare logit: the score scale does not apply)
   const float* sinks;
+  // span form only
+  int window, keep;          // window 0: none
+  int dk, dkp, dv;           // one map's key size, the key row's (maps * dk), value size
+  float cap_in, cap_log2;    // cap_in > 0: score -> cap * tanh(raw * scale / cap): cap_in = scale / cap, cap_log2 = cap * log2 e
+  float lam, eps, factor;    // two maps: rms_div(a1 - lam * a2) * factor
 };
 
 // MN-major (N contiguous) 128B-swizzled operand: rows are K (keys), 64 elements of N per 128-byte row;
@@ -179,7 +193,7 @@ __device__ __forceinline__ uint32_t pack2(float a, float b) {
 //                assembled page by page from the paged cache (tmap_k / tmap_v, one TMA box per page and 64-column
 //                chunk, addressed through the block table), which already holds this step's keys (rope_kv_write
 //                runs first).  Query i of a sequence sits at position ctx + i, ctx = seq_len - q_len.
-template <typename T, int D, bool PAGED, bool BIAS = false>
+template <typename T, int D, bool PAGED, bool BIAS = false, int MAPS = 0>
 __global__ void __launch_bounds__(kThreads, PCfg<D>::MIN_CTAS)
 attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_constant__ CUtensorMap tmap_k,
                     const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ PArgs a) {
@@ -187,6 +201,8 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
   constexpr int BN = C::BN;
   constexpr int DSUB = D / 64;   // 64-column (128-byte) sub-tiles along head_dim
   constexpr int NSUB = BN / 64;  // 64-key sub-tiles of P along the key dimension
+  constexpr bool SPAN = MAPS > 0;
+  constexpr int QT = MAPS == 2 ? BM / 2 : BM;   // queries per CTA
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   if (smem - smem_raw > C::ALIGN_SLACK) {
@@ -216,12 +232,21 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
   const int seq_start = a.cu_seqlens[seq];
   const int len = a.cu_seqlens[seq + 1] - seq_start;
   // heaviest (longest causal range) query tiles are scheduled first
-  const int q0 = (gridDim.x - 1 - blockIdx.x) * BM;  // first query (position within the sequence) of this CTA
+  const int q0 = (gridDim.x - 1 - blockIdx.x) * QT;  // first query (position within the sequence) of this CTA
   if (q0 >= len) return;           // uniform for the whole CTA
   const int kvh = head / (a.hq / a.hkv);
   const int ctx = PAGED ? a.seq_lens[seq] - len : 0;   // tokens already in the cache before this step's queries
-  const int kv_end = min(ctx + len, ctx + q0 + BM);     // causal: keys [0, kv_end)
-  const int n_tiles = (kv_end + BN - 1) / BN;
+  const int kv_end = min(ctx + len, ctx + q0 + QT);     // causal: keys [0, kv_end)
+  // window: the walk takes tiles 0 .. n_first - 1 (kept first tokens), then t_first .. (the first row's window on)
+  int t_first = 0, n_first = 0;
+  if constexpr (SPAN) {
+    if (a.window > 0) {
+      t_first = max(0, ctx + q0 - a.window + 1) / BN;
+      n_first = min((a.keep + BN - 1) / BN, t_first);
+    }
+  }
+  const int n_tiles = (kv_end + BN - 1) / BN - t_first + n_first;
+  auto key_tile = [&](int j) { return SPAN ? (j < n_first ? j : j - n_first + t_first) : j; };
 
   if (warp == 0 && lane == 0) {
     tma_prefetch_desc(&tmap);
@@ -258,7 +283,21 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
     // ===================== TMA producer (whole warp runs the loop, one elected lane issues) ===============
     {
       const uint64_t pol = l2_policy_evict_last();
-      if (elect_one()) {
+      const uint32_t k_tx = SPAN ? (uint32_t)((a.dkp + 63) / 64) * (BN * 128) : (uint32_t)C::K_BYTES;
+      const uint32_t v_tx = SPAN ? (uint32_t)((a.dv + 63) / 64) * (BN * 128) : (uint32_t)C::V_BYTES;
+      if (SPAN && elect_one()) {
+        mbar_arrive_expect_tx(bar_q, k_tx * (BM / BN));
+        // q as [token][head * maps + map][dk]: 64 x 64 boxes.  Two maps: the lower box is map 1, the upper one map 2 shifted by its
+        // columns' place in the key row; columns outside the map (negative or beyond dk) arrive as zeros
+#pragma unroll
+        for (int c = 0; c < DSUB; ++c)
+          if (c * 64 < a.dkp) {
+#pragma unroll
+            for (int h = 0; h < BM / BN; ++h)
+              tma_load_3d(sQ + c * (BM * 128) + h * (BN * 128), &tmap, bar_q, c * 64 - (MAPS == 2 ? h * a.dk : 0),
+                          MAPS == 2 ? head * 2 + h : head, seq_start + q0 + (MAPS == 2 ? 0 : h * BN), pol);
+          }
+      } else if (!SPAN && elect_one()) {
         mbar_arrive_expect_tx(bar_q, C::Q_BYTES);
         // the tensor-map box is [BN rows x 64 cols]; a 128-row Q sub-tile is BM / BN stacked boxes
         // (the 128B-swizzle pattern repeats every 8 rows, so stacked boxes form one contiguous tile)
@@ -276,16 +315,16 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
         const int row = seq_start + j * BN;
         mbar_wait(&bar_kempty[stage], phase ^ 1, 50);
         if (elect_one()) {
-          mbar_arrive_expect_tx(&bar_kfull[stage], C::K_BYTES);
+          mbar_arrive_expect_tx(&bar_kfull[stage], k_tx);
           if constexpr (PAGED) {
             // BN / page boxes per 64-column chunk; 8-row multiples keep the 128B-swizzle pattern contiguous
             const int* bt = a.block_tables + (int64_t)seq * a.max_blocks;
             for (int pg = 0; pg < BN / a.page; ++pg) {
-              const int bi = min(a.max_blocks - 1, (j * BN) / a.page + pg);
+              const int bi = min(a.max_blocks - 1, (key_tile(j) * BN) / a.page + pg);
               const int crow = (bt[bi] * a.hkv + kvh) * a.page;
 #pragma unroll
               for (int c = 0; c < DSUB; ++c)
-                tma_load_2d(sK + stage * C::K_BYTES + c * (BN * 128) + pg * a.page * 128, &tmap_k, &bar_kfull[stage], c * 64, crow, pol);
+                if (!SPAN || c * 64 < a.dkp) tma_load_2d(sK + stage * C::K_BYTES + c * (BN * 128) + pg * a.page * 128, &tmap_k, &bar_kfull[stage], c * 64, crow, pol);
             }
           } else {
 #pragma unroll
@@ -296,15 +335,15 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
         __syncwarp();
         mbar_wait(&bar_vempty[stage], phase ^ 1, 51);
         if (elect_one()) {
-          mbar_arrive_expect_tx(&bar_vfull[stage], C::V_BYTES);
+          mbar_arrive_expect_tx(&bar_vfull[stage], v_tx);
           if constexpr (PAGED) {
             const int* bt = a.block_tables + (int64_t)seq * a.max_blocks;
             for (int pg = 0; pg < BN / a.page; ++pg) {
-              const int bi = min(a.max_blocks - 1, (j * BN) / a.page + pg);
+              const int bi = min(a.max_blocks - 1, (key_tile(j) * BN) / a.page + pg);
               const int crow = (bt[bi] * a.hkv + kvh) * a.page;
 #pragma unroll
               for (int c = 0; c < DSUB; ++c)
-                tma_load_2d(sV + stage * C::V_BYTES + c * (BN * 128) + pg * a.page * 128, &tmap_v, &bar_vfull[stage], c * 64, crow, pol);
+                if (!SPAN || c * 64 < a.dv) tma_load_2d(sV + stage * C::V_BYTES + c * (BN * 128) + pg * a.page * 128, &tmap_v, &bar_vfull[stage], c * 64, crow, pol);
             }
           } else {
 #pragma unroll
@@ -338,7 +377,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
         for (int c = 0; c < DSUB; ++c)
 #pragma unroll
           for (int k = 0; k < 4; ++k)
-            umma_f16_ss(tS + (j & 1) * BN, umma_desc_k_sw128(q_addr + c * (BM * 128) + k * 32),
+            if (!SPAN || c * 64 + k * 16 < a.dkp) umma_f16_ss(tS + (j & 1) * BN, umma_desc_k_sw128(q_addr + c * (BM * 128) + k * 32),
                         umma_desc_k_sw128(k_addr + c * (BN * 128) + k * 32), idesc_s, (c | k) ? 1u : 0u);
         umma_commit(&bar_s[j & 1]);
         umma_commit(&bar_kempty[stage]);
@@ -349,7 +388,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
   } else if (warp == 6) {
     // ===================== PV issuer =====================
     const int fmt = a.dtype == LLMSS_BF16 ? 1 : 0;
-    const uint32_t idesc_o = idesc_f16(fmt, BM, D, 1);   // O += P V  : B (= V) is MN-major
+    const uint32_t idesc_o = idesc_f16(fmt, BM, SPAN ? (a.dv + 15) / 16 * 16 : D, 1);   // O += P V  : B (= V) is MN-major
     const uint32_t p_addr = smem_u32(sP), v_base = smem_u32(sV);
     int stage = 0;
     uint32_t phase = 0;
@@ -382,14 +421,15 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
     // ===================== softmax / correction / epilogue: one thread per query row =====================
     const int quarter = warp & 3;
     const int row = quarter * 32 + lane;         // query row within the tile == TMEM lane
-    const int qrow = q0 + row;                   // query index within this step's tokens of the sequence
+    const int qrow = q0 + (MAPS == 2 ? (row & 63) : row);   // query index within this step's tokens of the sequence
     const int qpos = ctx + qrow;                 // absolute position (== key index of the same token)
     const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
     float m_run = -INFINITY, l_run = 0.f;
+    const float scale_log2 = (SPAN && a.cap_in > 0.f) ? a.cap_log2 : a.scale_log2;
     for (int j = 0; j < n_tiles; ++j) {
       mbar_wait(&bar_s[j & 1], (j >> 1) & 1, 70);
       tcgen05_fence_after();
-      const int kbase = j * BN;
+      const int kbase = key_tile(j) * BN;
       const bool diag = (kbase + BN - 1) > ctx + q0;   // some key of this tile may lie above the diagonal
       // the whole S row lives in registers (one TMEM read): raw scores, masked on diagonal tiles
       float sc[BN];
@@ -419,7 +459,17 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
           for (int i = 0; i < BN; ++i) sc[i] += bt[min(max(d0 - i, 0), dmax)];
         }
       }
-      if (diag) {
+      if constexpr (SPAN) {
+        if (a.cap_in > 0.f) softcap_scores<BN>(sc, a.cap_in);
+        // some row's window starts inside or behind this tile, and not all of the tile is kept
+        const bool low = a.window > 0 && kbase < ctx + q0 + QT - a.window && kbase + BN > a.keep;
+        if (diag || low) {
+          const int hi = qpos - kbase, lo = a.window > 0 ? hi - a.window + 1 : -1, kp = a.keep - kbase;
+#pragma unroll
+          for (int i = 0; i < BN; ++i)
+            if (i > hi || (i < lo && i >= kp)) sc[i] = -INFINITY;
+        }
+      } else if (diag) {
 #pragma unroll
         for (int i = 0; i < BN; ++i)
           if (kbase + i > qpos) sc[i] = -INFINITY;
@@ -434,7 +484,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
       const float m_tile = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
       // Lazy running max (scale > 0: max commutes with scaling): keep the old reference unless this tile
       // exceeds it by more than 2^8 -- p stays <= 256, far inside fp32 / bf16 / fp16 range.
-      const float m_tile_s = m_tile * a.scale_log2;
+      const float m_tile_s = m_tile * scale_log2;
       const bool grow = (j == 0) || (m_tile_s > m_run + 8.0f);
       const float m_new = grow ? fmaxf(m_run, m_tile_s) : m_run;
       const float alpha = (j == 0 || !grow) ? 1.0f : ex2_approx(m_run - m_new);
@@ -456,7 +506,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
           float e0, e1;
-          ffma2(e0, e1, sc[c * 32 + i], sc[c * 32 + i + 1], a.scale_log2, a.scale_log2, neg_m, neg_m);
+          ffma2(e0, e1, sc[c * 32 + i], sc[c * 32 + i + 1], scale_log2, scale_log2, neg_m, neg_m);
           const float p0 = ex2_approx(e0);
           const float p1 = (C::FMA_EXP_EVERY > 0 && ((i >> 1) % (C::FMA_EXP_EVERY > 0 ? C::FMA_EXP_EVERY : 1)) == 0) ? ex2_fma(e1) : ex2_approx(e1);
           fadd2(la[(i >> 1) & 3], lb[(i >> 1) & 3], la[(i >> 1) & 3], lb[(i >> 1) & 3], p0, p1);
@@ -511,15 +561,60 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
     if constexpr (BIAS) {
       if (a.gate != nullptr && qrow < len) inv_l *= 1.0f / (1.0f + __expf(-a.gate[(int64_t)(seq_start + qrow) * a.ldg + head]));
     }
-    T* orow = reinterpret_cast<T*>(a.out) + (int64_t)(seq_start + qrow) * a.ldo + (int64_t)head * D;
+    const int dv = SPAN ? a.dv : D;
+    T* orow = reinterpret_cast<T*>(a.out) + (int64_t)(seq_start + qrow) * a.ldo + (int64_t)head * dv;
+    if constexpr (MAPS == 2) {
+      // every MMA has retired, so the K stages are free: [column][64 rows] of 32-bit values
+      float* xb = reinterpret_cast<float*>(sK) + (row & 63);
+      if (row >= 64) {
+        const float f = inv_l * a.lam;
+#pragma unroll 1
+        for (int c = 0; c * 32 < dv; ++c) {
+          uint32_t r[32];
+          tmem_ld_32x32b_x32(tO + lane_off + c * 32, r);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (c * 32 + i < dv) xb[(c * 32 + i) * 64] = __uint_as_float(r[i]) * f;
+        }
+      }
+      asm volatile("bar.sync 1, 128;" ::: "memory");      // the four softmax warps
+      if (row < 64) {
+        float ss = 0.f;
+#pragma unroll 1
+        for (int c = 0; c * 32 < dv; ++c) {
+          uint32_t r[32];
+          tmem_ld_32x32b_x32(tO + lane_off + c * 32, r);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (c * 32 + i < dv) {
+              const float o = fmaf(__uint_as_float(r[i]), inv_l, -xb[(c * 32 + i) * 64]);
+              ss = fmaf(o, o, ss);
+              xb[(c * 32 + i) * 64] = o;
+            }
+        }
+        const float rs = rsqrtf(ss / (float)dv + a.eps) * a.factor;
+        if (qrow < len) {
+          for (int c = 0; c < dv; c += 8) {
+            float f8[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) f8[i] = xb[(c + i) * 64] * rs;
+            *reinterpret_cast<uint4*>(orow + c) = pack8<T>(f8);
+          }
+        }
+      }
+    } else
 #pragma unroll 1
     for (int c = 0; c < D / 32; ++c) {
+      if (SPAN && c * 32 >= dv) break;
       uint32_t r[32];
       tmem_ld_32x32b_x32(tO + lane_off + c * 32, r);
       tmem_ld_wait();
       if (qrow < len) {
 #pragma unroll
         for (int q = 0; q < 4; ++q) {
+          if (SPAN && c * 32 + q * 8 >= dv) break;
           float f8[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) f8[i] = __uint_as_float(r[q * 8 + i]) * inv_l;
@@ -560,6 +655,20 @@ int launch_prefill(const CUtensorMap& tm, const CUtensorMap& tk, const CUtensorM
   auto kern = attn_prefill_kernel<T, D, PAGED, BIAS>;
   LLMSS_CHECK_CUDA(configured.ensure(kern, C::SMEM_BYTES));
   dim3 grid((max_seqlen + BM - 1) / BM, a.hq, num_seqs);
+  LLMSS_CHECK_CUDA(launch_pdl(kern, grid, dim3(kThreads), (size_t)C::SMEM_BYTES, stream, tm, tk, tv, a));
+  return 0;
+}
+
+template <typename T, int D, int MAPS>
+int launch_span(const CUtensorMap& tm, const CUtensorMap& tk, const CUtensorMap& tv, const PArgs& a, int num_seqs, int max_q,
+                cudaStream_t stream) {
+  using C = PCfg<D>;
+  static PerDeviceSmem configured;
+  auto kern = attn_prefill_kernel<T, D, true, false, MAPS>;
+  LLMSS_CHECK_CUDA(configured.ensure(kern, C::SMEM_BYTES));
+  constexpr int QT = MAPS == 2 ? BM / 2 : BM;
+  dim3 grid((max_q + QT - 1) / QT, a.hq, num_seqs);
+  LLMSS_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "attn_prefill_span: grid too large");
   LLMSS_CHECK_CUDA(launch_pdl(kern, grid, dim3(kThreads), (size_t)C::SMEM_BYTES, stream, tm, tk, tv, a));
   return 0;
 }
@@ -731,4 +840,79 @@ LLMSS_API int llmss_attn_prefill_paged_sink(const void* q, int64_t ldq, const vo
   LLMSS_REQUIRE(scale > 0.f && (bias_over_scale == nullptr || n_dist > 0), "attn_prefill_paged_sink: needs a positive scale");
   return prefill_paged_impl(q, ldq, k_cache, v_cache, block_tables, max_blocks, seq_lens, out, ldo, cu_q, num_seqs, max_q, total_q,
                             hq, hkv, d, block_size, num_blocks, scale, dtype, bias_over_scale, n_dist, gate, ldg, stream, sinks);
+}
+
+// Span form: causal attention over the paged cache with a sliding window (0: none) that keeps the first keep_first tokens,
+// soft-capped scores (cap 0: none) and maps = 1 / 2 query / key vectors per head.  q [total_q][hq * maps][dk] (row stride ldq),
+// K pages [num_blocks][hkv][block_size][maps * dk], V pages [num_blocks][hkv][block_size][dv].  maps = 1: out [total_q][hq * dv]
+// (row stride ldo) holds the attention outputs; maps = 2: rms_div(a1 - lam * a2) * factor per head.  dk and dv multiples of 8,
+// maps * dk and dv at most 256.
+LLMSS_API int llmss_attn_prefill_span(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
+                                      int max_blocks, const int* seq_lens, void* out, int64_t ldo, const int* cu_q, int num_seqs,
+                                      int max_q, int total_q, int hq, int hkv, int dk, int dv, int maps, int block_size, int num_blocks,
+                                      float scale, int window, int keep_first, float cap, float lam, float eps, float factor, int dtype,
+                                      cudaStream_t stream) {
+  LLMSS_REQUIRE(dtype == LLMSS_F16 || dtype == LLMSS_BF16, "attn_prefill_span: dtype must be f16/bf16");
+  LLMSS_REQUIRE(maps == 1 || maps == 2, "attn_prefill_span: %d maps", maps);
+  LLMSS_REQUIRE(dk > 0 && dv > 0 && dk % 8 == 0 && dv % 8 == 0 && maps * dk <= 256 && dv <= 256,
+                "attn_prefill_span: key size %d x %d / value size %d unsupported", maps, dk, dv);
+  LLMSS_REQUIRE(hq > 0 && hkv > 0 && hq % hkv == 0, "attn_prefill_span: bad head grouping hq=%d hkv=%d", hq, hkv);
+  LLMSS_REQUIRE(block_size == 16 || block_size == 32 || block_size == 64, "attn_prefill_span: block_size=%d unsupported (16/32/64)", block_size);
+  LLMSS_REQUIRE(scale > 0.f && window >= 0 && keep_first >= 0 && cap >= 0.f, "attn_prefill_span: bad scale, window or cap");
+  LLMSS_REQUIRE(ldo % 8 == 0 && ((uintptr_t)out % 16) == 0 && ((uintptr_t)q % 16) == 0 && ldq % 8 == 0 &&
+                    (((uintptr_t)k_cache | (uintptr_t)v_cache) % 16) == 0,
+                "attn_prefill_span: q / out / pages must be 16-byte aligned");
+  LLMSS_REQUIRE((int64_t)hq * maps * dk <= ldq, "attn_prefill_span: q columns exceed the row stride");
+  if (num_seqs == 0 || total_q == 0 || max_q == 0) return 0;
+  PFN_encodeTiled enc = get_encode();
+  LLMSS_REQUIRE(enc != nullptr, "attn_prefill: cuTensorMapEncodeTiled entry point not available");
+  CUtensorMap tm, tk, tv;
+  cuuint64_t dims[3] = {(cuuint64_t)dk, (cuuint64_t)hq * maps, (cuuint64_t)total_q};
+  cuuint64_t strides[2] = {(cuuint64_t)dk * 2, (cuuint64_t)ldq * 2};
+  cuuint32_t box[3] = {64, 1, 64};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = enc(&tm, dtype == LLMSS_BF16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 3, const_cast<void*>(q),
+                   dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
+                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  LLMSS_REQUIRE(r == CUDA_SUCCESS, "attn_prefill_span: q tensor map failed (CUresult %d)", (int)r);
+  const int64_t crow = (int64_t)num_blocks * hkv * block_size;
+  if (int e = encode_2d(&tk, k_cache, dtype, maps * dk, crow, maps * dk, block_size)) return e;
+  if (int e = encode_2d(&tv, v_cache, dtype, dv, crow, dv, block_size)) return e;
+  PArgs a;
+  memset(&a, 0, sizeof(a));
+  a.cu_seqlens = cu_q;
+  a.seq_lens = seq_lens;
+  a.block_tables = block_tables;
+  a.max_blocks = max_blocks;
+  a.page = block_size;
+  a.out = out;
+  a.ldo = ldo;
+  a.hq = hq;
+  a.hkv = hkv;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.dtype = dtype;
+  a.window = window < (1 << 30) ? window : 0;
+  a.keep = keep_first < (1 << 30) ? keep_first : (1 << 30);
+  a.dk = dk;
+  a.dkp = maps * dk;
+  a.dv = dv;
+  a.cap_in = cap > 0.f ? scale / cap : 0.f;
+  a.cap_log2 = cap * 1.4426950408889634f;
+  a.lam = lam;
+  a.eps = eps;
+  a.factor = factor;
+  const int d = maps * dk > dv ? maps * dk : dv;
+#define LLMSS_PS(T_, D_)                                                               \
+  return maps == 2 ? launch_span<T_, D_, 2>(tm, tk, tv, a, num_seqs, max_q, stream)    \
+                   : launch_span<T_, D_, 1>(tm, tk, tv, a, num_seqs, max_q, stream)
+  if (dtype == LLMSS_F16) {
+    if (d <= 64) LLMSS_PS(__half, 64);
+    if (d <= 128) LLMSS_PS(__half, 128);
+    LLMSS_PS(__half, 256);
+  } else {
+    if (d <= 64) LLMSS_PS(__nv_bfloat16, 64);
+    if (d <= 128) LLMSS_PS(__nv_bfloat16, 128);
+    LLMSS_PS(__nv_bfloat16, 256);
+  }
+#undef LLMSS_PS
 }

@@ -271,6 +271,45 @@ __device__ __forceinline__ void tma_load_2d(void* smem_dst, const void* map, uin
       "l"(map), "r"(smem_u32(bar)), "r"(c0), "r"(c1), "l"(policy)
       : "memory");
 }
+// 3-D tile load
+__device__ __forceinline__ void tma_load_3d(void* smem_dst, const void* map, uint64_t* bar, int c0, int c1, int c2,
+                                            uint64_t policy) {
+  asm volatile(
+      "cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes.L2::cache_hint"
+      " [%0], [%1, {%3, %4, %5}], [%2], %6;" ::"r"(smem_u32(smem_dst)),
+      "l"(map), "r"(smem_u32(bar)), "r"(c0), "r"(c1), "r"(c2), "l"(policy)
+      : "memory");
+}
+
+// ---------------------------------------------------------------- soft cap
+// tanh for soft-capped attention scores, 32-bit.  |x| <= 0.5: an odd polynomial of degree 9 fitted on that range (relative error
+// 1.1e-7 in 32-bit arithmetic, FMA pipe only); larger: 1 - 2 / (e^(2x) + 1) (absolute error of a few units in the last place of
+// 1, +-1 at the ends).  The caller picks the form for a whole tile of scores by their largest magnitude.
+__device__ __forceinline__ float tanh_small(float x) {
+  const float y = x * x;
+  float p = fmaf(y, 0.01715168f, -0.052994445f);
+  p = fmaf(y, p, 0.1332491f);
+  p = fmaf(y, p, -0.33333075f);
+  return fmaf(x * y, p, x);
+}
+__device__ __forceinline__ float tanh_any(float x) { return 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * x)); }
+// N raw scores of one row: s -> tanh(s * f); warp-uniform choice of the form
+template <int N>
+__device__ __forceinline__ void softcap_scores(float (&s)[N], float f) {
+  float m = 0.f;
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    s[i] *= f;
+    m = fmaxf(m, fabsf(s[i]));
+  }
+  if (__any_sync(0xffffffffu, m > 0.5f)) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) s[i] = tanh_any(s[i]);
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i) s[i] = tanh_small(s[i]);
+  }
+}
 
 // ---------------------------------------------------------------- tcgen05 / TMEM
 __device__ __forceinline__ void tmem_alloc(uint32_t* smem_dst, uint32_t ncols) {  // whole warp

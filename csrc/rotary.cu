@@ -150,7 +150,9 @@ template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
   __shared__ float cs[kMaxPairs], sn[kMaxPairs];
   const int64_t t = blockIdx.x;
-  token_angles(a.freq, a.n, a.positions[t], a.mag, cs, sn);
+  pdl_launch_dependents();
+  token_angles(a.freq, a.n, a.positions[t], a.mag, cs, sn);      // inputs of the step, not of the kernel in front
+  pdl_wait();
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int dk = a.dk, dv = a.dv, nq = a.hq * a.maps, nk = a.hkv * a.maps, row = a.maps * dk;
@@ -498,11 +500,10 @@ LLMSS_API int llmss_norm_rope_kv_write(const float* qkv, int64_t ld, int hq, int
   const bool vec = interleaved && dk % 4 == 0 && dk <= 128 * kNrVec && (hkv == 0 || dv % 4 == 0) && ld % 4 == 0 &&
                    ((((uintptr_t)qkv) | ((uintptr_t)q_w) | ((uintptr_t)k_w) | ((uintptr_t)k_cache) | ((uintptr_t)v_cache) | ((uintptr_t)q_out)) & 15) == 0;
   if (vec) {
-    LLMSS_BY_DTYPE(dtype, (norm_rope_kv_write_kernel<T, true><<<T_, 256, 0, stream>>>(a)));
+    LLMSS_BY_DTYPE(dtype, LLMSS_CHECK_CUDA(launch_pdl(norm_rope_kv_write_kernel<T, true>, dim3(T_), dim3(256), 0, stream, a)));
   } else {
-    LLMSS_BY_DTYPE(dtype, (norm_rope_kv_write_kernel<T, false><<<T_, 256, 0, stream>>>(a)));
+    LLMSS_BY_DTYPE(dtype, LLMSS_CHECK_CUDA(launch_pdl(norm_rope_kv_write_kernel<T, false>, dim3(T_), dim3(256), 0, stream, a)));
   }
-  LLMSS_CHECK_CUDA(cudaGetLastError());
   return 0;
 }
 

@@ -489,7 +489,7 @@ class RotaryAttention:
         with trace("norm_rope_kv_write"):
             q = ops.norm_rope_kv_write(y, H, G if self.own_kv else 0, D, Dv, self.maps, self.q_norm, self.k_norm, self.eps, self.freq,
                                        self.mag, self.interleaved, batch.positions, batch.slot_mapping, lc.k, lc.v, batch=batch,
-                                       out_dtype=dtype)
+                                       scale=self.scale, out_dtype=dtype)
         with trace("attention_window" if self.diff is None else "attention_diff"):
             return ops.attention_bias(q, lc.k, lc.v, batch, H, G, D, Dv, self.scale, None, out_dtype=dtype, window=self.window,
                                       keep_first=self.keep_first, softcap=self.softcap, diff=self.combine, out=out)

@@ -412,14 +412,15 @@ def residual_norm(resid, y, weight, bias, eps, kind, out_dtype=None):
 
 
 def norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, interleaved, positions, slot_mapping, k_cache, v_cache,
-                       batch=None, out_dtype=None):
+                       batch=None, scale=1.0, out_dtype=None):
     """Optional RMS norm with a weight per head (and map), rotation by a frequency table, keys and values to their pages; hkv = 0
-    prepares queries only.  ``batch`` lets the CUDA path lay the queries out for the attention kernel that will read them."""
+    prepares queries only.  ``batch`` and the score ``scale`` let the CUDA path lay the queries out for the attention kernel that will
+    read them (attention_bias with the same ``batch``)."""
     if _cuda(qkv):
         from . import cuda_impl as cu
 
         return cu.norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, interleaved, positions, slot_mapping, k_cache,
-                                     v_cache, batch, out_dtype)
+                                     v_cache, batch, scale, out_dtype)
     return ref.norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, interleaved, positions, slot_mapping, k_cache,
                                   v_cache, out_dtype)
 

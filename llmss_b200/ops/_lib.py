@@ -185,6 +185,12 @@ _SIGS = {
                                      c_float, c_int, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                                      c_int, c_void_p]),
     "llmss_diff_combine": (c_int, [c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p, c_int64, c_int, c_void_p]),
+    "llmss_attn_prefill_span": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int64, c_void_p,
+                                        c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
+                                        c_float, c_float, c_float, c_float, c_int, c_void_p]),
+    "llmss_attn_decode_span": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int64, c_void_p,
+                                       c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_float,
+                                       c_float, c_float, c_int, c_int, c_void_p]),
     "llmss_gated_simt": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int,
                                  c_void_p]),
 }

@@ -976,6 +976,28 @@ def attention_bias(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, dist_bias
 
 
 # --------------------------------------------------------------------------- windows with kept first tokens, soft cap, two maps per head
+_SPAN_TC = os.environ.get("LLMSS_ATTN_SPAN_TC", "1") == "1"
+
+
+def _span_tile(dk: int, dv: int, maps: int) -> int:
+    """Head size of the tensor-core tile that holds both the key row and the value (0: none does)."""
+    w = max(maps * dk, dv)
+    return 0 if w > 256 or dk % 8 or dv % 8 else (64 if w <= 64 else (128 if w <= 128 else 256))
+
+
+def span_uses_tc(dtype, dk: int, dv: int, maps: int, block_size: int, scale: float) -> bool:
+    """16-bit pages whose key and value sizes are multiples of 8 up to 256 run on the tcgen05 kernels; true 32-bit and everything
+    else on the generic one."""
+    return _SPAN_TC and dtype != torch.float32 and _span_tile(dk, dv, maps) > 0 and block_size in (16, 32, 64) and scale > 0
+
+
+def span_decode_uses_tc(dtype, hq: int, hkv: int, dk: int, dv: int, maps: int, block_size: int, scale: float) -> bool:
+    """The same for a batch of single tokens: the query heads of a group, times the maps, are the rows of one MMA tile.  Where
+    that tile does not fit, single tokens run on the prompt kernel."""
+    return (span_uses_tc(dtype, dk, dv, maps, block_size, scale) and hq * maps // hkv <= 128
+            and bool(_lib.load().llmss_attn_decode_tc_supported(hq * maps, hkv, _span_tile(dk, dv, maps), block_size)))
+
+
 def attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window=0, keep_first=0, softcap=0.0, diff=None, out_dtype=None,
                    out=None):
     """attention_bias without additive terms; see ops.reference.attention_bias for window, keep_first, softcap and diff."""
@@ -987,6 +1009,35 @@ def attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window=0,
     if out is None:
         out = torch.empty(T, hq * dv, dtype=dt, device=q.device)
     assert out.dtype == dt and out.shape == (T, hq * dv) and out.stride(1) == 1
+    lam, eps, factor = diff if diff is not None else (0.0, 0.0, 1.0)
+    if span_uses_tc(dt, dk, dv, maps, bs, scale):
+        if out.stride(0) % 8 or out.data_ptr() % 16:     # a view whose rows miss the kernels' 16-byte stores
+            return out.copy_(attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window, keep_first, softcap, diff, out_dtype))
+        assert q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
+        if q.shape[1] == hq * maps * maps * dk and batch.is_decode and span_decode_uses_tc(dt, hq, hkv, dk, dv, maps, bs, scale):
+            d = _span_tile(dk, dv, maps)
+            reach = min(batch.max_kv, window + keep_first + 128) if window else batch.max_kv
+            splits = decode_splits(batch.num_seqs, hq * maps, hkv, d, reach, dt, bs)
+            scratch = None
+            if splits > 1 or maps == 2:
+                scratch = arena(q.device).attn_scratch(lib.llmss_attn_decode_scratch_floats(T, hq * maps, d, splits), q.device)
+            rc = lib.llmss_attn_decode_span(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables),
+                                            batch.block_tables.shape[1], _ptr(batch.seq_lens), _ptr(out), out.stride(0), _ptr(scratch), T,
+                                            hq, hkv, dk, dv, maps, bs, k_cache.shape[0], float(scale), int(window), int(keep_first),
+                                            float(softcap), float(lam), float(eps), float(factor), splits, _DT[dt], _stream())
+            _lib.check(rc, "llmss_attn_decode_span")
+            _count(1 if splits == 1 and maps == 1 else 2)
+            return out
+        assert q.shape[1] == hq * maps * dk
+        rc = lib.llmss_attn_prefill_span(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables),
+                                         batch.block_tables.shape[1], _ptr(batch.seq_lens), _ptr(out), out.stride(0), _ptr(batch.cu_q),
+                                         batch.num_seqs, max(1, batch.max_q), T, hq, hkv, dk, dv, maps, bs, k_cache.shape[0], float(scale),
+                                         int(window), int(keep_first), float(softcap), float(lam), float(eps), float(factor), _DT[dt],
+                                         _stream())
+        _lib.check(rc, "llmss_attn_prefill_span")
+        _count()
+        return out
+    assert q.shape[1] == hq * maps * dk
     # the generic kernel: any sizes, true 32-bit; the two maps' outputs stay in 32-bit until they are combined
     o = torch.empty(T, hq * maps * dv, dtype=torch.float32, device=q.device) if maps == 2 else out
     rc = lib.llmss_attention_span(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables), batch.block_tables.shape[1],
@@ -996,7 +1047,6 @@ def attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window=0,
     _lib.check(rc, "llmss_attention_span")
     _count()
     if maps == 2:
-        lam, eps, factor = diff
         _lib.check(lib.llmss_diff_combine(_ptr(o), T, hq, dv, float(lam), float(eps), float(factor), _ptr(out), out.stride(0), _DT[dt],
                                           _stream()), "llmss_diff_combine")
         _count()
@@ -1022,15 +1072,19 @@ def residual_norm(resid, y, weight, bias, eps, kind, out_dtype=None):
 
 
 def norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, interleaved, positions, slot_mapping, k_cache, v_cache,
-                       batch=None, out_dtype=None):
+                       batch=None, scale=1.0, out_dtype=None):
+    """``batch``: a batch of single tokens whose attention (score ``scale``) will run on the tensor-core decode kernel gets its queries
+    as [T, hq * maps, maps * dk], zero outside the map's own columns."""
     lib = _lib.load()
     T, _, ld = _f32rows(qkv)
     dt = out_dtype or k_cache.dtype
     assert k_cache.dtype == dt and v_cache.dtype == dt and k_cache.is_contiguous() and v_cache.is_contiguous()
     assert k_cache.shape[3] == maps * dk and (hkv == 0 or (k_cache.shape[1] == hkv and v_cache.shape[3] == dv))
     assert all(w is None or (w.dtype == torch.float32 and w.numel() == dk) for w in (q_w, k_w))
-    pad = 0
-    q = torch.empty(T, hq * maps * dk, dtype=dt, device=qkv.device)
+    hkv_pages, bs = k_cache.shape[1], k_cache.shape[2]      # (hkv = 0: the pages are another layer's)
+    pad = int(maps > 1 and batch is not None and batch.is_decode
+              and span_decode_uses_tc(dt, hq, hkv_pages, dk, v_cache.shape[3], maps, bs, scale))
+    q = torch.empty(T, hq * maps * dk * (maps if pad else 1), dtype=dt, device=qkv.device)
     rc = lib.llmss_norm_rope_kv_write(_ptr(qkv), ld, hq, hkv, dk, dv, maps, _ptr(q_w), _ptr(k_w), float(eps),
                                       _ptr(_freq_dev(freq, qkv.device)), freq.numel(), float(mag), 1 if interleaved else 0, _ptr(positions),
                                       _ptr(slot_mapping), _ptr(k_cache), _ptr(v_cache), k_cache.shape[2], _ptr(q), pad, T, _DT[dt], _stream())

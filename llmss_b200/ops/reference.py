@@ -950,7 +950,9 @@ def softcap(z, cap: float):
 def residual_norm(resid, y, weight, bias, eps: float, kind: int, out_dtype=None):
     """norm_residual over a 32-bit residual stream: r = resid + y (y None: r = resid), h = LayerNorm or RMS norm of r.
     Returns (h in ``out_dtype``, r 32-bit)."""
-    h, r = norm_residual(resid, y, weight, bias, eps, kind, out_dtype=torch.float32)
+    h, r = norm_residual(resid, y, weight, bias if kind == NORM_LAYER else None, eps, kind, out_dtype=torch.float32)
+    if bias is not None and kind != NORM_LAYER:
+        h = h + bias.float()
     return h.to(out_dtype or torch.float32), r
 
 

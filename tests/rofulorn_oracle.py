@@ -147,3 +147,15 @@ def forward(tokens, cfg, p, return_layers=False):
         layers.append(x)
     logits = layer_norm(x, p["final.norm"], eps) @ p["head"].T
     return (logits, layers) if return_layers else logits
+
+
+def load_weights(path):
+    """Every tensor of a checkpoint folder in float64."""
+    from pathlib import Path
+
+    from safetensors.torch import load_file
+
+    out = {}
+    for f in sorted(Path(path).glob("*.safetensors")):
+        out.update({k: v.to(F64) for k, v in load_file(str(f)).items()})
+    return out
