@@ -299,19 +299,22 @@ template <typename T, int CH, int EPI, int ACT>
 __device__ __forceinline__ void store_chunk_full_t(const GemmArgs& a, const float (&v)[CH][8], int n, int mb0, int lane, float bval) {
   const bool has_res = a.residual != nullptr;
   if constexpr (EPI == EPI_GATED) {
-    // rows of w interleave (gate, up): even lane holds gate_j, odd lane up_j of output feature n/2
-    T* o = reinterpret_cast<T*>(a.out) + (int64_t)mb0 * a.ldo + (n >> 1);
-    const T* r = reinterpret_cast<const T*>(a.residual) + (int64_t)mb0 * a.ldr + (n >> 1);
-    const bool writer = (lane & 1) == 0;
+    // rows of w interleave (gate, up): even lane holds gate_j, odd lane up_j of output feature n/2.  Two token rows at a time: one
+    // exchange gives the even lane both numbers of the first row and the odd lane both of the second, so every lane applies
+    // the activation once and stores once
+    const int odd = lane & 1;
+    T* o = reinterpret_cast<T*>(a.out) + (int64_t)(mb0 + odd) * a.ldo + (n >> 1);
+    const T* r = reinterpret_cast<const T*>(a.residual) + (int64_t)(mb0 + odd) * a.ldr + (n >> 1);
 #pragma unroll
     for (int u = 0; u < CH; ++u)
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const float y = v[u][j] + bval;
-        const float other = __shfl_xor_sync(0xffffffffu, y, 1);
-        if (writer) *o = from_f32<T>(act_t<ACT>(y, a.act) * other + (has_res ? to_f32(*r) : 0.f));
-        o += a.ldo;
-        r += a.ldr;
+      for (int j = 0; j < 8; j += 2) {
+        const float y0 = v[u][j] + bval, y1 = v[u][j + 1] + bval;
+        const float got = __shfl_xor_sync(0xffffffffu, odd ? y0 : y1, 1);
+        const float gate = odd ? got : y0, up = odd ? y1 : got;
+        *o = from_f32<T>(act_t<ACT>(gate, a.act) * up + (has_res ? to_f32(*r) : 0.f));
+        o += 2 * a.ldo;
+        r += 2 * a.ldr;
       }
   } else {
     T* o = reinterpret_cast<T*>(a.out) + (int64_t)mb0 * a.ldo + n;

@@ -128,9 +128,10 @@ __global__ void __launch_bounds__(256) rope_norm_kv_write_kernel(const float* __
   }
 }
 
-// norm_rope_kv_write: grid T, block 256, a warp per vector of the token's row (hq * maps queries, hkv * maps keys, hkv values).
-// VEC: interleaved pairs and sizes that are multiples of four -- a lane holds its 4-column groups in registers from the 16-byte
-// load to the store; otherwise the row is re-read element by element.
+// norm_rope_kv_write: block 256, a warp per vector of the token's row (hq * maps queries, hkv * maps keys, hkv values).  Grid
+// (T, S): a decode batch spreads a token's vectors over S blocks, a prompt keeps them in one.  Vector form (interleaved pairs,
+// sizes that are multiples of four): a lane holds NV 4-column groups per vector in registers from the 16-byte load to the
+// store, and a warp's next P vectors are loaded before the first is worked on.  NV = 0: element by element, any size.
 struct NrArgs {
   const float* qkv; int64_t ld;
   int hq, hkv, dk, dv, maps;
@@ -142,11 +143,38 @@ struct NrArgs {
   void* q_out;
   int pad;                                // queries as [hq * maps][maps * dk], zero outside the map's own columns
 };
-constexpr int kNrVec = 4;                 // 4-column groups per lane: dk <= 512 in the vector form
+constexpr int kNrVec = 4;                 // most 4-column groups per lane: sizes up to 512 in the vector form
 
 template <typename T> struct alignas(4 * sizeof(T)) Quad { T v[4]; };
 
-template <typename T, bool VEC>
+// where vector u of the token goes (null: nowhere) and what it is
+template <typename T>
+__device__ __forceinline__ T* nr_target(const NrArgs& a, int64_t t, int u, int slot, int& width, const float*& w, int& map) {
+  const int nq = a.hq * a.maps, nk = a.hkv * a.maps, row = a.maps * a.dk;
+  w = nullptr;
+  width = a.dk;
+  map = -1;
+  if (u < nq) {
+    map = u % a.maps;
+    w = a.q_w;
+    return reinterpret_cast<T*>(a.q_out) + (a.pad ? (t * nq + u) * (int64_t)row + map * a.dk : (t * nq + u) * (int64_t)a.dk);
+  }
+  if (slot < 0) return nullptr;
+  const int64_t page = (int64_t)(slot / a.bs) * a.hkv * a.bs + slot % a.bs;      // row index of key/value head 0
+  if (u < nq + nk) {
+    map = (u - nq) % a.maps;
+    w = a.k_w;
+    return reinterpret_cast<T*>(a.k_cache) + (page + (int64_t)((u - nq) / a.maps) * a.bs) * row + map * a.dk;
+  }
+  width = a.dv;
+  return reinterpret_cast<T*>(a.v_cache) + (page + (int64_t)(u - nq - nk) * a.bs) * a.dv;
+}
+__device__ __forceinline__ const float* nr_source(const NrArgs& a, int64_t t, int u) {
+  const int n = (a.hq + a.hkv) * a.maps;
+  return a.qkv + t * a.ld + (u < n ? (int64_t)u * a.dk : (int64_t)n * a.dk + (int64_t)(u - n) * a.dv);
+}
+
+template <typename T, int NV>
 __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
   __shared__ float cs[kMaxPairs], sn[kMaxPairs];
   const int64_t t = blockIdx.x;
@@ -154,75 +182,80 @@ __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
   token_angles(a.freq, a.n, a.positions[t], a.mag, cs, sn);      // inputs of the step, not of the kernel in front
   pdl_wait();
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int dk = a.dk, dv = a.dv, nq = a.hq * a.maps, nk = a.hkv * a.maps, row = a.maps * dk;
+  const int warp = blockIdx.y * 8 + (threadIdx.x >> 5), warps = gridDim.y * 8, lane = threadIdx.x & 31;
+  const int dk = a.dk, nu = a.hq * a.maps + a.hkv * (a.maps + 1);
   const int slot = a.hkv > 0 ? a.slots[t] : -1;
-  const int64_t page = slot >= 0 ? (int64_t)(slot / a.bs) * a.hkv * a.bs + slot % a.bs : 0;    // row index of key/value head 0
-  T* kc = reinterpret_cast<T*>(a.k_cache);
-  T* vc = reinterpret_cast<T*>(a.v_cache);
-  for (int u = warp; u < nq + nk + a.hkv; u += 8) {
-    if (u >= nq && slot < 0) continue;
-    if (u >= nq + nk) {                                          // a value vector: as projected
-      const int g = u - nq - nk;
-      const float* x = a.qkv + t * a.ld + (int64_t)(nq + nk) * dk + (int64_t)g * dv;
-      T* dst = vc + (page + (int64_t)g * a.bs) * dv;
-      if constexpr (VEC) {
-        for (int c = lane * 4; c < dv; c += 128) {
-          const float4 v = *reinterpret_cast<const float4*>(x + c);
-          Quad<T> o{from_f32<T>(v.x), from_f32<T>(v.y), from_f32<T>(v.z), from_f32<T>(v.w)};
-          *reinterpret_cast<Quad<T>*>(dst + c) = o;
-        }
-      } else {
-        for (int c = lane; c < dv; c += 32) dst[c] = from_f32<T>(x[c]);
-      }
-      continue;
-    }
-    const bool is_q = u < nq;
-    const int hm = is_q ? u : u - nq, m = hm % a.maps;
-    const float* x = a.qkv + t * a.ld + (int64_t)u * dk;
-    const float* w = is_q ? a.q_w : a.k_w;
-    T* dst;
-    if (is_q) dst = reinterpret_cast<T*>(a.q_out) + (a.pad ? (t * nq + hm) * (int64_t)row + m * dk : (t * nq + hm) * (int64_t)dk);
-    else dst = kc + (page + (int64_t)(hm / a.maps) * a.bs) * row + m * dk;
-    if constexpr (VEC) {
-      float v[kNrVec][4];
-      float ss = 0.f;
+  if constexpr (NV > 0) {
+    constexpr int P = NV == 1 ? 4 : 1;
+    for (int u0 = warp; u0 < nu; u0 += warps * P) {
+      float v[P][NV > 0 ? NV : 1][4];
 #pragma unroll
-      for (int i = 0; i < kNrVec; ++i) {
-        const int c = lane * 4 + i * 128;
-        if (c < dk) {
-          const float4 f = *reinterpret_cast<const float4*>(x + c);
-          v[i][0] = f.x; v[i][1] = f.y; v[i][2] = f.z; v[i][3] = f.w;
-          ss = fmaf(f.x, f.x, fmaf(f.y, f.y, fmaf(f.z, f.z, fmaf(f.w, f.w, ss))));
+      for (int p = 0; p < P; ++p) {
+        const int u = u0 + p * warps;
+        if (u >= nu) continue;
+        const float* x = nr_source(a, t, u);
+        const int width = u < nu - a.hkv ? dk : a.dv;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int c = lane * 4 + i * 128;
+          float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (c < width) f = *reinterpret_cast<const float4*>(x + c);
+          v[p][i][0] = f.x; v[p][i][1] = f.y; v[p][i][2] = f.z; v[p][i][3] = f.w;
         }
       }
-      const float rstd = w != nullptr ? rsqrtf(warp_sum(ss) / (float)dk + a.eps) : 1.f;
 #pragma unroll
-      for (int i = 0; i < kNrVec; ++i) {
-        const int c = lane * 4 + i * 128;
-        if (c >= dk) continue;
+      for (int p = 0; p < P; ++p) {
+        const int u = u0 + p * warps;
+        if (u >= nu) continue;
+        int width, map;
+        const float* w;
+        T* dst = nr_target<T>(a, t, u, slot, width, w, map);
+        if (dst == nullptr) continue;
+        float rstd = 1.f;
         if (w != nullptr) {
-          const float4 wv = *reinterpret_cast<const float4*>(w + c);
-          v[i][0] *= rstd * wv.x; v[i][1] *= rstd * wv.y; v[i][2] *= rstd * wv.z; v[i][3] *= rstd * wv.w;
+          float ss = 0.f;
+#pragma unroll
+          for (int i = 0; i < NV; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) ss = fmaf(v[p][i][e], v[p][i][e], ss);
+          rstd = rsqrtf(warp_sum(ss) / (float)dk + a.eps);
         }
 #pragma unroll
-        for (int e = 0; e < 4; e += 2) {
-          const int pr = (c + e) >> 1;
-          if (pr < a.n) {
-            const float p = v[i][e], q = v[i][e + 1], cc = cs[pr], ssn = sn[pr];
-            v[i][e] = fmaf(p, cc, -q * ssn);
-            v[i][e + 1] = fmaf(q, cc, p * ssn);
+        for (int i = 0; i < NV; ++i) {
+          const int c = lane * 4 + i * 128;
+          if (c >= width) continue;
+          if (w != nullptr) {
+            const float4 wv = *reinterpret_cast<const float4*>(w + c);
+            v[p][i][0] *= rstd * wv.x; v[p][i][1] *= rstd * wv.y; v[p][i][2] *= rstd * wv.z; v[p][i][3] *= rstd * wv.w;
+          }
+          if (map >= 0) {
+#pragma unroll
+            for (int e = 0; e < 4; e += 2) {
+              const int pr = (c + e) >> 1;
+              if (pr < a.n) {
+                const float x0 = v[p][i][e], x1 = v[p][i][e + 1], cc = cs[pr], ssn = sn[pr];
+                v[p][i][e] = fmaf(x0, cc, -x1 * ssn);
+                v[p][i][e + 1] = fmaf(x1, cc, x0 * ssn);
+              }
+            }
+          }
+          const Quad<T> o{from_f32<T>(v[p][i][0]), from_f32<T>(v[p][i][1]), from_f32<T>(v[p][i][2]), from_f32<T>(v[p][i][3])};
+          *reinterpret_cast<Quad<T>*>(dst + c) = o;
+          if (a.pad && u < a.hq * a.maps) {                      // zeros where the other maps' columns are
+            const Quad<T> z{from_f32<T>(0.f), from_f32<T>(0.f), from_f32<T>(0.f), from_f32<T>(0.f)};
+            for (int m = 0; m < a.maps; ++m)
+              if (m != map) *reinterpret_cast<Quad<T>*>(dst + (m - map) * dk + c) = z;
           }
         }
-        Quad<T> o{from_f32<T>(v[i][0]), from_f32<T>(v[i][1]), from_f32<T>(v[i][2]), from_f32<T>(v[i][3])};
-        *reinterpret_cast<Quad<T>*>(dst + c) = o;
-        if (is_q && a.pad) {                                     // zeros where the other maps' columns are
-          const Quad<T> z{from_f32<T>(0.f), from_f32<T>(0.f), from_f32<T>(0.f), from_f32<T>(0.f)};
-          for (int o2 = 0; o2 < a.maps; ++o2)
-            if (o2 != m) *reinterpret_cast<Quad<T>*>(dst + (o2 - m) * dk + c) = z;
-        }
       }
-    } else {
+    }
+  } else {
+    for (int u = warp; u < nu; u += warps) {
+      int width, map;
+      const float* w;
+      T* dst = nr_target<T>(a, t, u, slot, width, w, map);
+      if (dst == nullptr) continue;
+      const float* x = nr_source(a, t, u);
       float rstd = 1.f;
       if (w != nullptr) {
         float ss = 0.f;
@@ -230,18 +263,18 @@ __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
         rstd = rsqrtf(warp_sum(ss) / (float)dk + a.eps);
       }
       auto normed = [&](int c) { return w != nullptr ? x[c] * (rstd * w[c]) : x[c]; };
-      for (int c = lane; c < dk; c += 32) {
+      for (int c = lane; c < width; c += 32) {
         float r = normed(c);
-        if (c < 2 * a.n) {
+        if (map >= 0 && c < 2 * a.n) {
           const bool second = a.interleaved ? (c & 1) : c >= a.n;
           const int pr = a.interleaved ? c >> 1 : (second ? c - a.n : c);
           const float o = normed(a.interleaved ? (c ^ 1) : (second ? c - a.n : c + a.n));
           r = second ? fmaf(r, cs[pr], o * sn[pr]) : fmaf(r, cs[pr], -o * sn[pr]);
         }
         dst[c] = from_f32<T>(r);
-        if (is_q && a.pad)
-          for (int o2 = 0; o2 < a.maps; ++o2)
-            if (o2 != m) dst[(o2 - m) * dk + c] = from_f32<T>(0.f);
+        if (a.pad && u < a.hq * a.maps)
+          for (int m = 0; m < a.maps; ++m)
+            if (m != map) dst[(m - map) * dk + c] = from_f32<T>(0.f);
       }
     }
   }
@@ -497,12 +530,17 @@ LLMSS_API int llmss_norm_rope_kv_write(const float* qkv, int64_t ld, int hq, int
   if (T_ <= 0) return 0;
   NrArgs a{qkv, ld, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, n_pairs, mag, interleaved, positions, slots, k_cache, v_cache,
            block_size, q_out, pad};
-  const bool vec = interleaved && dk % 4 == 0 && dk <= 128 * kNrVec && (hkv == 0 || dv % 4 == 0) && ld % 4 == 0 &&
+  const int widest = hkv > 0 && dv > dk ? dv : dk;
+  const bool vec = interleaved && dk % 4 == 0 && widest <= 128 * kNrVec && (hkv == 0 || dv % 4 == 0) && ld % 4 == 0 &&
                    ((((uintptr_t)qkv) | ((uintptr_t)q_w) | ((uintptr_t)k_w) | ((uintptr_t)k_cache) | ((uintptr_t)v_cache) | ((uintptr_t)q_out)) & 15) == 0;
-  if (vec) {
-    LLMSS_BY_DTYPE(dtype, LLMSS_CHECK_CUDA(launch_pdl(norm_rope_kv_write_kernel<T, true>, dim3(T_), dim3(256), 0, stream, a)));
+  const int rounds = (hq * maps + hkv * (maps + 1) + 7) / 8;          // vectors per warp if a token had one block
+  const dim3 grid(T_, T_ >= 1024 ? 1 : (rounds < 64 ? rounds : 64));
+  if (vec && widest <= 128) {
+    LLMSS_BY_DTYPE(dtype, LLMSS_CHECK_CUDA(launch_pdl(norm_rope_kv_write_kernel<T, 1>, grid, dim3(256), 0, stream, a)));
+  } else if (vec) {
+    LLMSS_BY_DTYPE(dtype, LLMSS_CHECK_CUDA(launch_pdl(norm_rope_kv_write_kernel<T, kNrVec>, grid, dim3(256), 0, stream, a)));
   } else {
-    LLMSS_BY_DTYPE(dtype, LLMSS_CHECK_CUDA(launch_pdl(norm_rope_kv_write_kernel<T, false>, dim3(T_), dim3(256), 0, stream, a)));
+    LLMSS_BY_DTYPE(dtype, LLMSS_CHECK_CUDA(launch_pdl(norm_rope_kv_write_kernel<T, 0>, grid, dim3(256), 0, stream, a)));
   }
   return 0;
 }

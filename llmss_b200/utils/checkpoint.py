@@ -520,15 +520,15 @@ def _rofulorn_shapes(cfg: dict):
 
 
 def _rofulorn_preset(width, vocab, heads, ff, n_blocks, window=1024, kv_div=4):
-    """``n_blocks`` x (plain, differential, plain, differential on the pages of the block's second layer), each with a gated
-    feed-forward; head size 128 (plain) and 2 x 64 over values of 128 (differential)."""
+    """``n_blocks`` x (plain, differential, plain), every layer with a gated feed-forward; the differential layer of every second
+    block attends over the pages of the one before.  Head size 128 (plain), 2 x 64 over values of 128 (differential)."""
     G = max(1, heads // kv_div)
     pln = dict(type="attention_2", heads=heads, kv_heads=G, dim=128, vdim=128, rot_dims=64, base=500000.0, window=window, mlp={"ff": ff})
     dif = dict(type="attention", heads=heads, kv_heads=G, dim=64, vdim=128, rot_dims=32, window=2 * window, keep_first=8, diff=0.45,
                softcap=30.0, scaling={"factor": 4.0, "low": 1.0, "high": 4.0, "original": 4096}, mlp={"ff": ff})
     layers = []
     for b in range(n_blocks):
-        layers += [dict(pln), dict(dif), dict(pln), dict(dif, kv_from=4 * b + 1)]
+        layers += [dict(pln), dict(dif, kv_from=3 * b - 2) if b % 2 else dict(dif), dict(pln)]
     return rofulorn_config(width, vocab, layers, embed_scale=width ** 0.5)
 
 
@@ -539,9 +539,10 @@ PRESETS.update({
         dict(type="attention_2", heads=4, kv_heads=1, dim=32, vdim=24, rot_dims=24, window=33, mlp={"ff": 160}),
         dict(type="attention", heads=6, kv_heads=2, dim=24, vdim=40, rot_dims=16, window=12, keep_first=5, diff=0.7, kv_from=0, mlp=None)],
         embed_scale=8.0),
-    # sizes whose layers resemble a served model's (random weights), beside gptj-like-* of equal width and depth
-    "rofulorn-2k": _rofulorn_preset(2048, 32000, 16, 6144, 5),
-    "rofulorn-4k": _rofulorn_preset(4096, 32000, 32, 10240, 4),
+    # sizes whose layers resemble a served model's (random weights), beside gptj-like-* of equal width and depth; three feed-forward
+    # matrices of these sizes hold about as many weights as the two of gptj-like-*
+    "rofulorn-2k": _rofulorn_preset(2048, 32000, 16, 2816, 6),
+    "rofulorn-4k": _rofulorn_preset(4096, 32000, 32, 4096, 6),
 })
 
 
