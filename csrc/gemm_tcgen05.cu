@@ -368,7 +368,7 @@ __device__ __forceinline__ void cluster_sync_all() {
   asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
-// execution-only rendezvous of the cluster (no memory ordering: no MEMBAR / cache invalidation in the SASS)
+// execution-only rendezvous of the cluster (relaxed: no memory ordering)
 __device__ __forceinline__ void cluster_sync_relaxed() {
   asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
@@ -515,7 +515,7 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
     // ===================== epilogue (4 warps = 128 TMEM lanes) =====================
     // The accumulator is consumed in groups of 8 token columns through *rolled* loops: the
     // epilogue runs once per segment, so its code must stay small enough not to be
-    // instruction-fetch bound (a fully unrolled 256-column epilogue is ~20k SASS instructions).
+    // instruction-fetch bound (a fully unrolled 256-column epilogue is).
     const int quarter = warp & 3;            // TMEM lane quarter this warp may access
     const int f = quarter * 32 + lane;       // feature within the tile
     const int epi_tid = threadIdx.x - 64;
