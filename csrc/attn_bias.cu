@@ -22,7 +22,8 @@
 
 namespace {
 
-constexpr int NW = 8, TK = 32, MAXV = 8;   // warps per CTA, keys per tile, output channels per lane (dv <= 256)
+constexpr int NW = 8, TK = 32;             // warps per CTA, keys per tile
+constexpr int MAXV_ALL = 16;               // most output channels per lane (dv <= 512); kernels are instantiated for 8 and 16
 
 template <typename T>
 __global__ void __launch_bounds__(256) qknorm_kv_write_kernel(const float* __restrict__ qkv, int64_t ld, int hq, int hkv, int dk,
@@ -144,7 +145,7 @@ struct AbArgs {
   float cap;                              // > 0: scaled score s -> cap * tanh(s / cap), before bias and slopes
 };
 
-template <typename T, typename TO>
+template <typename T, typename TO, int MAXV>
 __global__ void __launch_bounds__(NW * 32) attention_bias_kernel(AbArgs a) {
   extern __shared__ float sm[];
   const int b = blockIdx.z;
@@ -256,9 +257,9 @@ __global__ void __launch_bounds__(256) diff_combine_kernel(const float* __restri
   const int lane = threadIdx.x & 31;
   const float* a1 = x + u * 2 * dv;
   const float* a2 = a1 + dv;
-  float v[MAXV], ss = 0.f;
+  float v[MAXV_ALL], ss = 0.f;
 #pragma unroll
-  for (int i = 0; i < MAXV; ++i) {
+  for (int i = 0; i < MAXV_ALL; ++i) {
     const int c = lane + 32 * i;
     v[i] = c < dv ? fmaf(-lam, a2[c], a1[c]) : 0.f;
     ss = fmaf(v[i], v[i], ss);
@@ -266,7 +267,7 @@ __global__ void __launch_bounds__(256) diff_combine_kernel(const float* __restri
   const float r = rsqrtf(warp_sum(ss) / (float)dv + eps) * factor;
   T* o = out + (u / hq) * ldo + (u % hq) * dv;
 #pragma unroll
-  for (int i = 0; i < MAXV; ++i) {
+  for (int i = 0; i < MAXV_ALL; ++i) {
     const int c = lane + 32 * i;
     if (c < dv) o[c] = from_f32<T>(v[i] * r);
   }
@@ -324,7 +325,7 @@ static int attention_bias_launch(const void* q, int64_t ldq, const void* k_cache
                                  const float* sinks = nullptr, int maps = 1, int keep = 0, float cap = 0.f, int64_t ldo = 0,
                                  int out_f32 = 0) {
   LLMSS_REQUIRE(hq > 0 && hkv > 0 && hq % hkv == 0, "attention_bias: %d query heads over %d key/value heads", hq, hkv);
-  LLMSS_REQUIRE(dv <= 32 * MAXV, "attention_bias: value size %d (at most %d)", dv, 32 * MAXV);
+  LLMSS_REQUIRE(dv <= 32 * MAXV_ALL, "attention_bias: value size %d (at most %d)", dv, 32 * MAXV_ALL);
   LLMSS_REQUIRE(bias == nullptr || n_dist > 0, "attention_bias: empty bias table");
   if (B <= 0 || max_q <= 0) return 0;
   AbArgs a;
@@ -343,9 +344,9 @@ static int attention_bias_launch(const void* q, int64_t ldq, const void* k_cache
   LLMSS_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "attention_bias: grid too large");
 #define LLMSS_AB(TT, TO)                                                                \
   do {                                                                              \
-    static PerDeviceSmem gsm;                                                       \
-    auto kern = attention_bias_kernel<TT, TO>;                                      \
-    LLMSS_CHECK_CUDA(gsm.ensure(kern, (int)smem));                                  \
+    static PerDeviceSmem gsm[2];                                                    \
+    auto kern = dv <= 256 ? attention_bias_kernel<TT, TO, 8> : attention_bias_kernel<TT, TO, 16>; \
+    LLMSS_CHECK_CUDA(gsm[dv <= 256 ? 0 : 1].ensure(kern, (int)smem));               \
     kern<<<grid, NW * 32, smem, stream>>>(a);                                       \
   } while (0)
   if (dtype == LLMSS_F16 && out_f32) LLMSS_AB(__half, float);
@@ -404,7 +405,7 @@ LLMSS_API int llmss_attention_span(const void* q, int64_t ldq, const void* k_cac
 // x [T][hq][2][dv] 32-bit -> out [T][hq * dv] (row stride ldo): rms_div(x1 - lam * x2) * factor per head
 LLMSS_API int llmss_diff_combine(const float* x, int T_, int hq, int dv, float lam, float eps, float factor, void* out, int64_t ldo,
                                  int dtype, cudaStream_t stream) {
-  LLMSS_REQUIRE(hq > 0 && dv > 0 && dv <= 32 * MAXV, "diff_combine: value size %d (at most %d)", dv, 32 * MAXV);
+  LLMSS_REQUIRE(hq > 0 && dv > 0 && dv <= 32 * MAXV_ALL, "diff_combine: value size %d (at most %d)", dv, 32 * MAXV_ALL);
   if (T_ <= 0) return 0;
   const int64_t units = (int64_t)T_ * hq;
   LLMSS_BY_DTYPE(dtype, (diff_combine_kernel<T><<<(unsigned)((units + NW - 1) / NW), NW * 32, 0, stream>>>(x, hq, dv, lam, eps, factor,

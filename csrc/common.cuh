@@ -281,33 +281,55 @@ __device__ __forceinline__ void tma_load_3d(void* smem_dst, const void* map, uin
       : "memory");
 }
 
+// ---------------------------------------------------------------- packed arithmetic
+// Packed fp32x2 arithmetic (one issue slot for two numbers): the softmax warps of the prompt-attention kernel are bound by
+// instruction issue (ncu: issue 50 %, tensor pipe 45 % before this), so the scale-and-shift, the row-sum and the soft cap run
+// on it.
+__device__ __forceinline__ void ffma2(float& d0, float& d1, float a0, float a1, float b0, float b1, float c0, float c1) {
+  asm("{\n\t.reg .b64 a, b, c, d;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmov.b64 c, {%6, %7};\n\t"
+      "fma.rn.f32x2 d, a, b, c;\n\tmov.b64 {%0, %1}, d;\n\t}"
+      : "=f"(d0), "=f"(d1) : "f"(a0), "f"(a1), "f"(b0), "f"(b1), "f"(c0), "f"(c1));
+}
+__device__ __forceinline__ void fadd2(float& d0, float& d1, float a0, float a1, float b0, float b1) {
+  asm("{\n\t.reg .b64 a, b, d;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tadd.rn.f32x2 d, a, b;\n\tmov.b64 {%0, %1}, d;\n\t}"
+      : "=f"(d0), "=f"(d1) : "f"(a0), "f"(a1), "f"(b0), "f"(b1));
+}
+
+__device__ __forceinline__ void fmul2(float& d0, float& d1, float a0, float a1, float b0, float b1) {
+  asm("{\n\t.reg .b64 a, b, d;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmul.rn.f32x2 d, a, b;\n\tmov.b64 {%0, %1}, d;\n\t}"
+      : "=f"(d0), "=f"(d1) : "f"(a0), "f"(a1), "f"(b0), "f"(b1));
+}
+
 // ---------------------------------------------------------------- soft cap
 // tanh for soft-capped attention scores, 32-bit.  |x| <= 0.5: an odd polynomial of degree 9 fitted on that range (relative error
 // 1.1e-7 in 32-bit arithmetic, FMA pipe only); larger: 1 - 2 / (e^(2x) + 1) (absolute error of a few units in the last place of
 // 1, +-1 at the ends).  The caller picks the form for a whole tile of scores by their largest magnitude.
-__device__ __forceinline__ float tanh_small(float x) {
-  const float y = x * x;
-  float p = fmaf(y, 0.01715168f, -0.052994445f);
-  p = fmaf(y, p, 0.1332491f);
-  p = fmaf(y, p, -0.33333075f);
-  return fmaf(x * y, p, x);
+__device__ __forceinline__ void tanh_small2(float& x0, float& x1) {
+  float y0, y1, p0, p1;
+  fmul2(y0, y1, x0, x1, x0, x1);
+  ffma2(p0, p1, y0, y1, 0.01715168f, 0.01715168f, -0.052994445f, -0.052994445f);
+  ffma2(p0, p1, y0, y1, p0, p1, 0.1332491f, 0.1332491f);
+  ffma2(p0, p1, y0, y1, p0, p1, -0.33333075f, -0.33333075f);
+  fmul2(y0, y1, x0, x1, y0, y1);
+  ffma2(x0, x1, y0, y1, p0, p1, x0, x1);
 }
 __device__ __forceinline__ float tanh_any(float x) { return 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * x)); }
 // N raw scores of one row: s -> tanh(s * f); warp-uniform choice of the form
 template <int N>
 __device__ __forceinline__ void softcap_scores(float (&s)[N], float f) {
-  float m = 0.f;
+  static_assert(N % 4 == 0, "rows of whole pairs");
+  float m[2] = {0.f, 0.f};
 #pragma unroll
-  for (int i = 0; i < N; ++i) {
-    s[i] *= f;
-    m = fmaxf(m, fabsf(s[i]));
+  for (int i = 0; i < N; i += 2) {
+    fmul2(s[i], s[i + 1], s[i], s[i + 1], f, f);
+    m[(i >> 1) & 1] = fmaxf(m[(i >> 1) & 1], fmaxf(fabsf(s[i]), fabsf(s[i + 1])));
   }
-  if (__any_sync(0xffffffffu, m > 0.5f)) {
+  if (__any_sync(0xffffffffu, fmaxf(m[0], m[1]) > 0.5f)) {
 #pragma unroll
     for (int i = 0; i < N; ++i) s[i] = tanh_any(s[i]);
   } else {
 #pragma unroll
-    for (int i = 0; i < N; ++i) s[i] = tanh_small(s[i]);
+    for (int i = 0; i < N; i += 2) tanh_small2(s[i], s[i + 1]);
   }
 }
 

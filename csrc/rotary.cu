@@ -130,8 +130,9 @@ __global__ void __launch_bounds__(256) rope_norm_kv_write_kernel(const float* __
 
 // norm_rope_kv_write: block 256, a warp per vector of the token's row (hq * maps queries, hkv * maps keys, hkv values).  Grid
 // (T, S): a decode batch spreads a token's vectors over S blocks, a prompt keeps them in one.  Vector form (interleaved pairs,
-// sizes that are multiples of four): a lane holds NV 4-column groups per vector in registers from the 16-byte load to the
-// store, and a warp's next P vectors are loaded before the first is worked on.  NV = 0: element by element, any size.
+// sizes that are multiples of four): LPV lanes share a vector (16: short ones, two per warp) and hold NV 4-column groups each in
+// registers from the 16-byte load to the store; the next P vectors are loaded before the first is worked on.  NV = 0: element
+// by element, any size.
 struct NrArgs {
   const float* qkv; int64_t ld;
   int hq, hkv, dk, dv, maps;
@@ -174,7 +175,7 @@ __device__ __forceinline__ const float* nr_source(const NrArgs& a, int64_t t, in
   return a.qkv + t * a.ld + (u < n ? (int64_t)u * a.dk : (int64_t)n * a.dk + (int64_t)(u - n) * a.dv);
 }
 
-template <typename T, int NV>
+template <typename T, int NV, int LPV>
 __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
   __shared__ float cs[kMaxPairs], sn[kMaxPairs];
   const int64_t t = blockIdx.x;
@@ -186,18 +187,20 @@ __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
   const int dk = a.dk, nu = a.hq * a.maps + a.hkv * (a.maps + 1);
   const int slot = a.hkv > 0 ? a.slots[t] : -1;
   if constexpr (NV > 0) {
-    constexpr int P = NV == 1 ? 4 : 1;
-    for (int u0 = warp; u0 < nu; u0 += warps * P) {
+    constexpr int P = NV <= 2 ? 4 / NV : 1, VPW = 32 / LPV;
+    const int sub = lane / LPV, l4 = (lane % LPV) * 4, step = warps * VPW;
+    const uint32_t mates = LPV == 32 ? 0xffffffffu : (uint32_t)((1u << (LPV & 31)) - 1u) << (sub * LPV);
+    for (int u0 = warp * VPW + sub; u0 < nu; u0 += step * P) {
       float v[P][NV > 0 ? NV : 1][4];
 #pragma unroll
       for (int p = 0; p < P; ++p) {
-        const int u = u0 + p * warps;
+        const int u = u0 + p * step;
         if (u >= nu) continue;
         const float* x = nr_source(a, t, u);
         const int width = u < nu - a.hkv ? dk : a.dv;
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
-          const int c = lane * 4 + i * 128;
+          const int c = l4 + i * (LPV * 4);
           float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
           if (c < width) f = *reinterpret_cast<const float4*>(x + c);
           v[p][i][0] = f.x; v[p][i][1] = f.y; v[p][i][2] = f.z; v[p][i][3] = f.w;
@@ -205,7 +208,7 @@ __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
       }
 #pragma unroll
       for (int p = 0; p < P; ++p) {
-        const int u = u0 + p * warps;
+        const int u = u0 + p * step;
         if (u >= nu) continue;
         int width, map;
         const float* w;
@@ -218,11 +221,13 @@ __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
           for (int i = 0; i < NV; ++i)
 #pragma unroll
             for (int e = 0; e < 4; ++e) ss = fmaf(v[p][i][e], v[p][i][e], ss);
-          rstd = rsqrtf(warp_sum(ss) / (float)dk + a.eps);
+#pragma unroll
+          for (int o = LPV / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(mates, ss, o);
+          rstd = rsqrtf(ss / (float)dk + a.eps);
         }
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
-          const int c = lane * 4 + i * 128;
+          const int c = l4 + i * (LPV * 4);
           if (c >= width) continue;
           if (w != nullptr) {
             const float4 wv = *reinterpret_cast<const float4*>(w + c);
@@ -533,15 +538,18 @@ LLMSS_API int llmss_norm_rope_kv_write(const float* qkv, int64_t ld, int hq, int
   const int widest = hkv > 0 && dv > dk ? dv : dk;
   const bool vec = interleaved && dk % 4 == 0 && widest <= 128 * kNrVec && (hkv == 0 || dv % 4 == 0) && ld % 4 == 0 &&
                    ((((uintptr_t)qkv) | ((uintptr_t)q_w) | ((uintptr_t)k_w) | ((uintptr_t)k_cache) | ((uintptr_t)v_cache) | ((uintptr_t)q_out)) & 15) == 0;
-  const int rounds = (hq * maps + hkv * (maps + 1) + 7) / 8;          // vectors per warp if a token had one block
+  const bool half = dk <= 64 && widest <= 128;                          // 16 lanes per vector
+  const int per = half ? 16 : 8;
+  const int rounds = (hq * maps + hkv * (maps + 1) + per - 1) / per;    // vectors per warp (half) if a token had one block
   const dim3 grid(T_, T_ >= 1024 ? 1 : (rounds < 64 ? rounds : 64));
-  if (vec && widest <= 128) {
-    LLMSS_BY_DTYPE(dtype, LLMSS_CHECK_CUDA(launch_pdl(norm_rope_kv_write_kernel<T, 1>, grid, dim3(256), 0, stream, a)));
-  } else if (vec) {
-    LLMSS_BY_DTYPE(dtype, LLMSS_CHECK_CUDA(launch_pdl(norm_rope_kv_write_kernel<T, kNrVec>, grid, dim3(256), 0, stream, a)));
-  } else {
-    LLMSS_BY_DTYPE(dtype, LLMSS_CHECK_CUDA(launch_pdl(norm_rope_kv_write_kernel<T, 0>, grid, dim3(256), 0, stream, a)));
-  }
+#define LLMSS_NR(NV_, LPV_) \
+  LLMSS_BY_DTYPE(dtype, LLMSS_CHECK_CUDA(launch_pdl(norm_rope_kv_write_kernel<T, NV_, LPV_>, grid, dim3(256), 0, stream, a)))
+  if (vec && half && widest <= 64) LLMSS_NR(1, 16);
+  else if (vec && half) LLMSS_NR(2, 16);
+  else if (vec && widest <= 128) LLMSS_NR(1, 32);
+  else if (vec) LLMSS_NR(kNrVec, 32);
+  else LLMSS_NR(0, 32);
+#undef LLMSS_NR
   return 0;
 }
 

@@ -402,6 +402,43 @@ int llmss_bgemm_simt_ex(const void* x, int64_t ldx, int64_t sxh, const void* w, 
                         int64_t soh, int M, int N, int K, int H, int act, int act_start, int dtype, int out_f32,
                         llmss_stream_t stream);
 
+/* ---- parallel sub-layers over a 32-bit residual, windows with kept first tokens, soft-capped scores, two maps per head */
+/* out_r = resid + y (y null: out_r null, nothing stored); out_h = LayerNorm (kind 0) or RMS norm (kind 1) of it times weight
+ * (+ bias), weights 32-bit */
+int llmss_residual_norm(const float* resid, int64_t ldr, const float* y, int64_t ldy, const float* weight, const float* bias,
+                        float* out_r, void* out_h, int M, int W, float eps, int kind, int out_dtype, llmss_stream_t stream);
+/* qkv [T][hq*maps*dk | hkv*maps*dk | hkv*dv] 32-bit: q, k vectors rms-normed with weight q_w / k_w [dk] (null: no norm), rotated, k to
+ * the K pages [.., maps * dk], v as it is to the V pages; q_out [T][hq*maps][dk], or [..][maps*dk] zero-padded (pad = 1); hkv = 0:
+ * queries only */
+int llmss_norm_rope_kv_write(const float* qkv, int64_t ld, int hq, int hkv, int dk, int dv, int maps, const float* q_w,
+                             const float* k_w, float eps, const double* freq, int n_pairs, float mag, int interleaved,
+                             const int* positions, const int* slots, void* k_cache, void* v_cache, int block_size, void* q_out,
+                             int pad, int T, int dtype, llmss_stream_t stream);
+/* generic attention: window > 0 hides keys with i - j >= window unless j < keep_first; cap > 0: cap tanh(s / cap); maps vectors
+ * per head side by side in the key row (hq counts heads x maps) */
+int llmss_attention_span(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
+                         int max_blocks, int block_size, const int* seq_lens, const int* cu_q, int window, int keep_first, float cap,
+                         int maps, void* out, int64_t ldo, int out_f32, int B, int max_q, int hq, int hkv, int dk, int dv, float scale,
+                         int dtype, llmss_stream_t stream);
+/* x [T][hq][2][dv] 32-bit -> out [T][hq * dv]: rms_div(x1 - lam x2) * factor per head */
+int llmss_diff_combine(const float* x, int T, int hq, int dv, float lam, float eps, float factor, void* out, int64_t ldo, int dtype,
+                       llmss_stream_t stream);
+/* the same attention on the tcgen05 kernels (16-bit; dk, dv multiples of 8, maps * dk and dv <= 256; maps 1 or 2, hq counts heads;
+ * maps = 2: out is the combination).  Prompt portions: q [total_q][hq * maps][dk]; single tokens: q [B][hq * maps][maps * dk],
+ * zero-padded, scratch of llmss_attn_decode_scratch_floats(B, hq * maps, 64 / 128 / 256, num_splits) floats */
+int llmss_attn_prefill_span(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
+                            int max_blocks, const int* seq_lens, void* out, int64_t ldo, const int* cu_q, int num_seqs, int max_q,
+                            int total_q, int hq, int hkv, int dk, int dv, int maps, int block_size, int num_blocks, float scale,
+                            int window, int keep_first, float cap, float lam, float eps, float factor, int dtype,
+                            llmss_stream_t stream);
+int llmss_attn_decode_span(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
+                           int max_blocks, const int* seq_lens, void* out, int64_t ldo, float* scratch, int B, int hq, int hkv, int dk,
+                           int dv, int maps, int block_size, int num_blocks, float scale, int window, int keep_first, float cap,
+                           float lam, float eps, float factor, int num_splits, int dtype, llmss_stream_t stream);
+/* out[t][n] = act(x_t . w_2n) * (x_t . w_2n+1) on the CUDA cores (any size, 32-bit or 16-bit) */
+int llmss_gated_simt(const void* x, int64_t ldx, const void* w, int64_t ldw, const void* bias, void* out, int64_t ldo, int M,
+                     int n_out, int K, int act, int dtype, llmss_stream_t stream);
+
 #ifdef __cplusplus
 }
 #endif

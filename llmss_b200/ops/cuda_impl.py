@@ -888,9 +888,9 @@ from .reference import window_bias_table  # noqa: E402  (the window and slopes a
 
 def attention_bias(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, dist_bias, gate=None, out_dtype=None, bias_over_scale=None,
                    window=0, slopes=None, sinks=None, keep_first=0, softcap=0.0, diff=None, dst=None):
-    if keep_first or softcap or diff is not None or dst is not None or (window and slopes is None and dist_bias is None):
-        assert dist_bias is None and slopes is None and gate is None and sinks is None, \
-            "attention: kept first tokens, soft cap and two-map heads have no bias, slopes, gate or sink beside them"
+    plain = dist_bias is None and slopes is None and gate is None and sinks is None
+    if plain or keep_first or softcap or diff is not None or dst is not None:
+        assert plain, "attention: kept first tokens, soft cap and two-map heads have no bias, slopes, gate or sink beside them"
         return attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window or 0, keep_first, softcap, diff, out_dtype, dst)
     lib = _lib.load()
     T = q.shape[0]

@@ -32,7 +32,7 @@ def test_loaded_library_is_the_in_tree_one():
 
 
 @pytest.mark.parametrize("H,G,dk,dv,maps,cap", [(4, 2, 8, 12, 1, 0.0), (4, 2, 8, 12, 2, 9.0), (3, 3, 6, 10, 2, 0.0), (2, 1, 20, 5, 1, 12.0),
-                                                (18, 1, 40, 72, 2, 20.0), (4, 2, 136, 24, 1, 0.0)])
+                                                (18, 1, 40, 72, 2, 20.0), (4, 2, 136, 24, 1, 0.0), (2, 1, 12, 300, 2, 4.0)])
 def test_generic_attention(H, G, dk, dv, maps, cap):
     cases.test_window_edges_first_tokens_and_far_keys(H, G, dk, dv, maps, cap, "cuda", F32, 1e-4, bs=64)
     cases.test_window_edges_first_tokens_and_far_keys(H, G, dk, dv, maps, cap, "cuda", F32, 1e-4, bs=16, spans=[(20, 4), (33, 20)])
