@@ -94,11 +94,13 @@ __device__ __forceinline__ int balanced_quota(int total_tiles, int grid) {
   return (total_tiles + active - 1) / active > 1 ? (total_tiles + active - 1) / active : 1;
 }
 
+template <bool SPAN>
 __device__ __forceinline__ int key_tile(const Item& r, int j) {
   const int v = r.v_begin + j;
-  return v < r.n_first ? v : v - r.n_first + r.t_first;
+  return SPAN && v >= r.n_first ? v - r.n_first + r.t_first : v;
 }
 
+template <bool SPAN, int BN>
 __device__ __forceinline__ Item decode_item(const DArgs& a, int it) {
   Item r;
   const int split = it % a.num_splits;
@@ -106,9 +108,9 @@ __device__ __forceinline__ Item decode_item(const DArgs& a, int it) {
   r.kvh = t % a.hkv;
   r.b = t / a.hkv;
   r.L = a.seq_lens[r.b];
-  r.t_first = a.window > 0 ? max(0, r.L - a.window) / a.bn : 0;
-  r.n_first = min((a.keep + a.bn - 1) / a.bn, r.t_first);
-  const int total = r.L > 0 ? (r.L + a.bn - 1) / a.bn - r.t_first + r.n_first : 0;
+  r.t_first = SPAN && a.window > 0 ? max(0, r.L - a.window) / BN : 0;
+  r.n_first = SPAN ? min((a.keep + BN - 1) / BN, r.t_first) : 0;
+  const int total = r.L > 0 ? (r.L + BN - 1) / BN - r.t_first + r.n_first : 0;
   const int chunk = (total + a.num_splits - 1) / a.num_splits;  // whole key tiles per split
   r.v_begin = split * chunk;
   r.n_tiles = max(0, min(total - r.v_begin, chunk));
@@ -124,11 +126,12 @@ __device__ __forceinline__ Item decode_item(const DArgs& a, int it) {
 //    contiguous ranges, one per CTA ("stream-K" for attention): a CTA's range may start and end in the
 //    middle of an item, those pieces are written as partials and merged by the combine kernel.  Removes
 //    the wave quantisation of items / SMs (e.g. 128 items on 148 SMs at TP=8).
+template <bool SPAN, int BN>
 struct Sched {
   const DArgs& a;
   int it;                             // split mode cursor
   int t, t_stop, b, kvh, j, quota;    // balanced mode cursor: flat tile index, (sequence, kv head, tile)
-  __device__ __forceinline__ int ntiles(int i) const { return (a.seq_lens[i] + a.bn - 1) / a.bn; }
+  __device__ __forceinline__ int ntiles(int i) const { return (a.seq_lens[i] + BN - 1) / BN; }
   __device__ Sched(const DArgs& a_) : a(a_), it(blockIdx.x), t(0), t_stop(0), b(0), kvh(0), j(0), quota(1) {
     if (!a.balanced) return;
     int total = 0;
@@ -154,7 +157,7 @@ struct Sched {
   __device__ bool next(Item& r) {
     if (!a.balanced) {
       if (it >= a.n_items) return false;
-      r = decode_item(a, it);
+      r = decode_item<SPAN, BN>(a, it);
       it += gridDim.x;
       return true;
     }
@@ -256,7 +259,7 @@ __device__ __forceinline__ void softmax_bar(int threads) { asm volatile("bar.syn
 // MUFU) would do all the exponentials.  Replicating the rows R times lets the warps of copy c handle the
 // key columns [c * 64 / R, (c + 1) * 64 / R) of the same heads: the row max is agreed through shared
 // memory once per tile, P rows are assembled in shared memory by all copies, l is summed at the end.
-template <typename T, int D, int R>
+template <typename T, int D, int R, bool SPAN>
 __global__ void __launch_bounds__(kThreads, 1)
 attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                       const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ DArgs a) {
@@ -291,6 +294,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int G = a.G;
+  const int dk = SPAN ? a.dk : D, dv = SPAN ? a.dv : D;     // key row and value size (the plain form: the tile's)
   pdl_launch_dependents();
   constexpr int QPC = 4 / R;  // softmax warps (TMEM lane quarters) per copy
   int n_live_warps = 0;
@@ -334,18 +338,18 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
     const int pages = BN / a.block_size;
     int stage = 0, n = 0;
     uint32_t phase = 0;
-    Sched sch(a);
+    Sched<SPAN, BN> sch(a);
     Item I;
     while (sch.next(I)) {
       if (I.n_tiles == 0) continue;
       const int qb = n & 1;
       mbar_wait(&bar_qempty[qb], ((n >> 1) & 1) ^ 1, 40);
       if (elect_one()) {
-        mbar_arrive_expect_tx(&bar_qfull[qb], (uint32_t)(a.q_copies * a.q_box_rows * ((a.dk + 63) / 64) * 128));
+        mbar_arrive_expect_tx(&bar_qfull[qb], (uint32_t)(a.q_copies * a.q_box_rows * ((dk + 63) / 64) * 128));
         for (int cc = 0; cc < a.q_copies; ++cc)
 #pragma unroll
           for (int c = 0; c < DSUB; ++c)
-            if (c * 64 < a.dk) tma_load_3d(sQ + qb * q_bytes + c * q_chunk + cc * (a.q_box_rows * 128), &tmap_q, &bar_qfull[qb], c * 64,
+            if (c * 64 < dk) tma_load_3d(sQ + qb * q_bytes + c * q_chunk + cc * (a.q_box_rows * 128), &tmap_q, &bar_qfull[qb], c * 64,
                         I.kvh * G, I.b, pol_q);
       }
       // Block-table entries are fetched 32 pages at a time (one coalesced load per warp, the next group
@@ -355,7 +359,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
       const int last_page = (I.L - 1) / bs;
       const int tiles_per_group = 32 / pages;
       auto load_rows = [&](int group) {
-        const int pg = key_tile(I, group * tiles_per_group + lane / pages) * pages + lane % pages;
+        const int pg = SPAN ? key_tile<SPAN>(I, group * tiles_per_group + lane / pages) * pages + lane % pages
+                            : I.v_begin * pages + group * 32 + lane;
         // pages past the end of the sequence are masked later: fetch the reserved block 0 instead
         const int blk = (pg <= last_page) ? __ldg(bt + pg) : 0;
         return (blk * a.hkv + I.kvh) * bs;
@@ -368,21 +373,21 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
           if (j + tiles_per_group < I.n_tiles) nxt = load_rows(j / tiles_per_group + 1);
         }
         mbar_wait(&bar_kempty[stage], phase ^ 1, 50);
-        if (elect_one()) mbar_arrive_expect_tx(&bar_kfull[stage], (uint32_t)a.k_tx);
+        if (elect_one()) mbar_arrive_expect_tx(&bar_kfull[stage], SPAN ? (uint32_t)a.k_tx : (uint32_t)KV_BYTES);
         __syncwarp();
         for (int p = 0; p < pages; ++p) {
           const int row = __shfl_sync(0xffffffffu, cur, tg * pages + p);
           if (elect_one())
-            for (int c = 0; c < a.k_ops; ++c)
+            for (int c = 0; c < (SPAN ? a.k_ops : 1); ++c)
               tma_load_3d(sK + stage * KV_BYTES + p * (bs * D * 2) + c * (bs * 128), &tmap_k, &bar_kfull[stage], c * 64, row, 0, pol_kv);
         }
         mbar_wait(&bar_vempty[stage], phase ^ 1, 51);
-        if (elect_one()) mbar_arrive_expect_tx(&bar_vfull[stage], (uint32_t)a.v_tx);
+        if (elect_one()) mbar_arrive_expect_tx(&bar_vfull[stage], SPAN ? (uint32_t)a.v_tx : (uint32_t)KV_BYTES);
         __syncwarp();
         for (int p = 0; p < pages; ++p) {
           const int row = __shfl_sync(0xffffffffu, cur, tg * pages + p);
           if (elect_one())
-            for (int c = 0; c < a.v_ops; ++c)
+            for (int c = 0; c < (SPAN ? a.v_ops : 1); ++c)
               tma_load_3d(sV + stage * KV_BYTES + p * (bs * D * 2) + c * (bs * 128), &tmap_v, &bar_vfull[stage], c * 64, row, 0, pol_kv);
         }
         if (++stage == S) { stage = 0; phase ^= 1; }
@@ -404,7 +409,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
     const uint32_t page_bytes = bs * D * 2, chunk_bytes = bs * 128;
     int kst = 0, n = 0;
     uint32_t kph = 0, g = 0;
-    Sched sch(a);
+    Sched<SPAN, BN> sch(a);
     Item I;
     while (sch.next(I)) {
       if (I.n_tiles == 0) continue;
@@ -423,7 +428,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
             for (int c = 0; c < DSUB; ++c)
 #pragma unroll
               for (int k = 0; k < 4; ++k)
-                if (c * 64 + k * 16 < a.dk) umma_f16_ss_ws(tS + (g & 1) * 16, umma_desc_k_sw128_sbo(q_addr + c * q_chunk + k * 32, a.q_sbo),
+                if (c * 64 + k * 16 < dk) umma_f16_ss_ws(tS + (g & 1) * 16, umma_desc_k_sw128_sbo(q_addr + c * q_chunk + k * 32, a.q_sbo),
                                umma_desc_k_sw128(k_addr + c * chunk_bytes + k * 32), idesc_ws, (c | k) ? 1u : 0u);
             umma_commit(&bar_s[g & 1]);
             umma_commit(&bar_kempty[kst]);
@@ -435,7 +440,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
             for (int c = 0; c < DSUB; ++c)
 #pragma unroll
               for (int k = 0; k < 4; ++k)
-                if (c * 64 + k * 16 < a.dk) umma_f16_ss(tS + (g & 1) * BN + p * bs, umma_desc_k_sw128_sbo(q_addr + c * q_chunk + k * 32, a.q_sbo),
+                if (c * 64 + k * 16 < dk) umma_f16_ss(tS + (g & 1) * BN + p * bs, umma_desc_k_sw128_sbo(q_addr + c * q_chunk + k * 32, a.q_sbo),
                             umma_desc_k_sw128(k_addr + p * page_bytes + c * chunk_bytes + k * 32), idesc_s,
                             (c | k) ? 1u : 0u);
           umma_commit(&bar_s[g & 1]);
@@ -456,7 +461,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
     const uint32_t page_bytes = bs * D * 2, chunk_bytes = bs * 128;
     int vst = 0;
     uint32_t vph = 0, g = 0;
-    Sched sch(a);
+    Sched<SPAN, BN> sch(a);
     Item I;
     while (sch.next(I)) {
       for (int j = 0; j < I.n_tiles; ++j, ++g) {
@@ -501,8 +506,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
     const int n_threads = n_live_warps * 32;
     const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
     uint32_t g = 0;
-    const float scale_log2 = a.cap_in > 0.f ? a.cap_log2 : a.scale_log2;
-    Sched sch(a);
+    const float scale_log2 = SPAN && a.cap_in > 0.f ? a.cap_log2 : a.scale_log2;
+    Sched<SPAN, BN> sch(a);
     Item I;
     while (sch.next(I)) {
       const int head = I.kvh * G + row;
@@ -510,8 +515,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
       if (I.n_tiles == 0) {  // empty split (or empty sequence): neutral partial / zero output
         if (live && owner) {
           if (I.direct) {
-            T* orow = reinterpret_cast<T*>(a.out) + (int64_t)I.b * a.ldo + (int64_t)head * a.dv;
-            for (int c = 0; c < a.dv; c += 8) *reinterpret_cast<uint4*>(orow + c) = make_uint4(0, 0, 0, 0);
+            T* orow = reinterpret_cast<T*>(a.out) + (int64_t)I.b * a.ldo + (int64_t)head * dv;
+            for (int c = 0; c < dv; c += 8) *reinterpret_cast<uint4*>(orow + c) = make_uint4(0, 0, 0, 0);
           } else {
             for (int c = 0; c < D; c += 4) *reinterpret_cast<float4*>(a.part_o + pidx * D + c) = make_float4(0, 0, 0, 0);
             a.part_ml[pidx * 2] = -INFINITY;
@@ -524,7 +529,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
       for (int j = 0; j < I.n_tiles; ++j, ++g) {
         mbar_wait(&bar_s[g & 1], (g >> 1) & 1, 70);
         tcgen05_fence_after();
-        const int kbase = key_tile(I, j) * BN + c0;
+        const int kbase = key_tile<SPAN>(I, j) * BN + c0;
         float sc[CW];
         if constexpr (CW == 16) {
           uint32_t r[16];
@@ -546,13 +551,13 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
         tcgen05_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(&bar_sfree[g & 1]);  // S(g) is in registers: the buffer can take QK(g+2)
-        if (a.cap_in > 0.f) softcap_scores<CW>(sc, a.cap_in);
+        if (SPAN && a.cap_in > 0.f) softcap_scores<CW>(sc, a.cap_in);
         if (kbase + CW > I.L) {
 #pragma unroll
           for (int i = 0; i < CW; ++i)
             if (kbase + i >= I.L) sc[i] = -INFINITY;
         }
-        if (a.window > 0 && kbase < I.L - a.window && kbase + CW > a.keep) {   // the window starts inside or behind these keys
+        if (SPAN && a.window > 0 && kbase < I.L - a.window && kbase + CW > a.keep) {   // the window starts inside or behind these keys
           const int lo = I.L - a.window - kbase, kp = a.keep - kbase;
 #pragma unroll
           for (int i = 0; i < CW; ++i)
@@ -647,10 +652,10 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
         tmem_ld_wait();
         if (!live) continue;
         if (I.direct) {
-          T* orow = reinterpret_cast<T*>(a.out) + (int64_t)I.b * a.ldo + (int64_t)head * a.dv + e_base;
+          T* orow = reinterpret_cast<T*>(a.out) + (int64_t)I.b * a.ldo + (int64_t)head * dv + e_base;
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
-            if (e_base + c * 32 + q * 8 >= a.dv) break;
+            if (e_base + c * 32 + q * 8 >= dv) break;
             float f8[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) f8[i] = __uint_as_float(r[q * 8 + i]) * inv_l;
@@ -813,11 +818,11 @@ int plan_stages(int q_alloc_rows, int d, int* smem_bytes) {
   return stages;
 }
 
-template <typename T, int D, int R>
+template <typename T, int D, int R, bool SPAN>
 int launch_decode_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const DArgs& a, int smem,
                      cudaStream_t stream) {
   static PerDeviceSmem configured;
-  auto kern = attn_decode_tc_kernel<T, D, R>;
+  auto kern = attn_decode_tc_kernel<T, D, R, SPAN>;
   LLMSS_CHECK_CUDA(configured.ensure(kern, smem));
   const int grid = (a.balanced || a.n_items >= sm_count()) ? sm_count() : a.n_items;
   LLMSS_CHECK_CUDA(launch_pdl(kern, dim3(grid), dim3(kThreads), (size_t)smem, stream, tq, tk, tv, a));
@@ -982,11 +987,14 @@ static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const
     a.partials = span->maps > 1 ? 1 : 0;
   }
   int rc = 0;
-#define LLMSS_DT(T_, D_)                                                         \
-  do {                                                                           \
-    if (R == 4) rc = launch_decode_tc<T_, D_, 4>(tq, tk, tv, a, smem, stream);      \
-    else if (R == 2) rc = launch_decode_tc<T_, D_, 2>(tq, tk, tv, a, smem, stream); \
-    else rc = launch_decode_tc<T_, D_, 1>(tq, tk, tv, a, smem, stream);             \
+#define LLMSS_DT_(T_, D_, R_)                                                                  \
+  rc = span != nullptr ? launch_decode_tc<T_, D_, R_, true>(tq, tk, tv, a, smem, stream)       \
+                       : launch_decode_tc<T_, D_, R_, false>(tq, tk, tv, a, smem, stream)
+#define LLMSS_DT(T_, D_)                    \
+  do {                                      \
+    if (R == 4) LLMSS_DT_(T_, D_, 4);       \
+    else if (R == 2) LLMSS_DT_(T_, D_, 2);  \
+    else LLMSS_DT_(T_, D_, 1);              \
   } while (0)
   if (dtype == LLMSS_F16) {
     if (d == 64) LLMSS_DT(__half, 64);
@@ -998,6 +1006,7 @@ static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const
     else LLMSS_DT(__nv_bfloat16, 256);
   }
 #undef LLMSS_DT
+#undef LLMSS_DT_
   if (rc != 0 || (num_splits == 1 && a.partials == 0)) return rc;
   if (span != nullptr) {
     const dim3 cgrid(hq / span->maps, B);
