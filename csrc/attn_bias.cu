@@ -9,9 +9,9 @@
 //                     its warps share every 32-key tile of K and V, staged once in shared memory in 32-bit.  A warp owns
 //                     one pair: lane = key inside the tile for the scores, lane = output channel (mod 32) for P V.
 //                     Scores, softmax and accumulation are 32-bit with full-precision exponentials.
-//                     Optional: a linear penalty slopes[h] * (i - j) taken off the scores, and a sliding window (keys with
-//                     i - j >= window are hidden; the key loop starts at the first row's window) that may keep the sequence's
-//                     first tokens, soft-capped scores cap * tanh(s / cap), and two query / key maps per head side by side in
+//                     Optional: a linear penalty slopes[h] * (i - j) taken off the scores, a sliding window (keys with
+//                     i - j >= window are hidden; the key loop starts at the first row's window) or a chunked mask (only keys of
+//                     the query's own block of positions), either of which may keep the sequence's first tokens, soft-capped scores cap * tanh(s / cap), and two query / key maps per head side by side in
 //                     the key row (the values are the head's; one output per map).
 //   diff_combine    : the two maps' outputs of a head -> rms_div(a1 - lam * a2) * factor.
 //   qkv_prepare     : the general form of qknorm_kv_write, one CTA per token: query / key norm per head or over the token's
@@ -143,6 +143,8 @@ struct AbArgs {
   int maps;                               // query heads h = head * maps + map read columns [map * dk, (map + 1) * dk) of the key row
   int keep;                               // with a window: keys j < keep are visible whatever their distance
   float cap;                              // > 0: scaled score s -> cap * tanh(s / cap), before bias and slopes
+  int chunk;                              // > 0: only keys of the query's own block of `chunk` positions are visible
+  int ldv;                                // row stride of the V pages (>= dv)
 };
 
 template <typename T, typename TO, int MAXV>
@@ -179,8 +181,8 @@ __global__ void __launch_bounds__(NW * 32) attention_bias_kernel(AbArgs a) {
   const T* vc = reinterpret_cast<const T*>(a.v_cache);
   const float* brow = a.bias != nullptr ? a.bias + (int64_t)(active ? h : 0) * a.n_dist : nullptr;
   const float slope = a.slopes != nullptr && active ? a.slopes[h] : 0.f;
-  const int kbeg = a.window > 0 ? max(0, ctx + r0 - a.window + 1) : 0;      // first key any row of this CTA sees
-  const int klo = a.window > 0 ? qpos - a.window + 1 : 0;                   // first key of this warp's row's window
+  const int kbeg = first_visible(ctx + r0, a.window, a.chunk);              // first key any row of this CTA sees
+  const int klo = first_visible(qpos, a.window, a.chunk);                   // first key this warp's row sees
   const int kfirst = min(a.keep, kbeg);                                     // kept keys in front of the window: [0, kfirst)
   const int kcol = a.maps > 1 ? (h % a.maps) * dk : 0;
   int k1 = 0;                                                               // end of the tile = start of the next one
@@ -196,7 +198,7 @@ __global__ void __launch_bounds__(NW * 32) attention_bias_kernel(AbArgs a) {
     for (int idx = threadIdx.x; idx < nk * dv; idx += NW * 32) {
       const int kk = idx / dv, c = idx % dv, pos = k0 + kk;
       const int blk = a.block_tables[(int64_t)b * a.max_blocks + pos / a.bs];
-      vs[kk * dv + c] = to_f32(vc[(((int64_t)blk * a.hkv + g) * a.bs + pos % a.bs) * dv + c]);
+      vs[kk * dv + c] = to_f32(vc[(((int64_t)blk * a.hkv + g) * a.bs + pos % a.bs) * a.ldv + c]);
     }
     __syncthreads();
     if (!active || k0 > qpos || (k1 <= klo && k0 >= a.keep)) continue;
@@ -323,7 +325,7 @@ static int attention_bias_launch(const void* q, int64_t ldq, const void* k_cache
                                  int n_dist, const float* slopes, int window, const float* gate, int64_t ldg, void* out, int B,
                                  int max_q, int hq, int hkv, int dk, int dv, float scale, int dtype, cudaStream_t stream,
                                  const float* sinks = nullptr, int maps = 1, int keep = 0, float cap = 0.f, int64_t ldo = 0,
-                                 int out_f32 = 0) {
+                                 int out_f32 = 0, int chunk = 0, int ldv = 0) {
   LLMSS_REQUIRE(hq > 0 && hkv > 0 && hq % hkv == 0, "attention_bias: %d query heads over %d key/value heads", hq, hkv);
   LLMSS_REQUIRE(dv <= 32 * MAXV_ALL, "attention_bias: value size %d (at most %d)", dv, 32 * MAXV_ALL);
   LLMSS_REQUIRE(bias == nullptr || n_dist > 0, "attention_bias: empty bias table");
@@ -334,6 +336,7 @@ static int attention_bias_launch(const void* q, int64_t ldq, const void* k_cache
   a.sinks = sinks;
   a.hq = hq; a.hkv = hkv; a.dk = dk; a.dv = dv; a.scale = scale;
   a.maps = maps; a.keep = keep; a.cap = cap; a.ldo = ldo > 0 ? ldo : (int64_t)hq * dv;
+  a.chunk = chunk; a.ldv = ldv > 0 ? ldv : dv;
   const int gsz = hq / hkv;
   a.nh = gsz < NW ? gsz : NW;
   a.rows = NW / a.nh;
@@ -392,14 +395,27 @@ LLMSS_API int llmss_attention_sink(const void* q, int64_t ldq, const void* k_cac
 // the same with everything at once: a window that keeps the sequence's first `keep_first` tokens, soft-capped scores (cap > 0) and
 // `maps` query / key vectors per head (hq counts heads x maps: query head h is map h % maps; key rows are maps * dk wide, the
 // key / value head of query head h is h / (hq / hkv)).  out [T][hq * dv] with row stride ldo, 32-bit if out_f32.
+// chunk > 0: only keys of the query's own block of `chunk` positions; sinks [hq] or null; ldv: row stride of the V pages (the value may
+// be the leading columns of a wider row).
+LLMSS_API int llmss_attention_span_ex(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, int ldv,
+                                      const int* block_tables, int max_blocks, int block_size, const int* seq_lens, const int* cu_q,
+                                      int window, int chunk, int keep_first, float cap, int maps, const float* sinks, void* out,
+                                      int64_t ldo, int out_f32, int B, int max_q, int hq, int hkv, int dk, int dv, float scale, int dtype,
+                                      cudaStream_t stream) {
+  LLMSS_REQUIRE(chunk >= 0 && ldv >= dv, "attention_span: chunk %d, value rows of %d for %d columns", chunk, ldv, dv);
+  LLMSS_REQUIRE(window >= 0 && keep_first >= 0 && cap >= 0.f && maps >= 1 && hkv > 0 && (hq / hkv) % maps == 0,
+                "attention_span: window %d, keep_first %d, cap %f, %d maps, %d query heads", window, keep_first, cap, maps, hq);
+  return attention_bias_launch(q, ldq, k_cache, v_cache, block_tables, max_blocks, block_size, seq_lens, cu_q, nullptr, 0, nullptr, window,
+                               nullptr, 0, out, B, max_q, hq, hkv, dk, dv, scale, dtype, stream, sinks, maps, keep_first, cap, ldo, out_f32,
+                               chunk, ldv);
+}
+
 LLMSS_API int llmss_attention_span(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
                                    int max_blocks, int block_size, const int* seq_lens, const int* cu_q, int window, int keep_first,
                                    float cap, int maps, void* out, int64_t ldo, int out_f32, int B, int max_q, int hq, int hkv, int dk,
                                    int dv, float scale, int dtype, cudaStream_t stream) {
-  LLMSS_REQUIRE(window >= 0 && keep_first >= 0 && cap >= 0.f && maps >= 1 && hkv > 0 && (hq / hkv) % maps == 0,
-                "attention_span: window %d, keep_first %d, cap %f, %d maps, %d query heads", window, keep_first, cap, maps, hq);
-  return attention_bias_launch(q, ldq, k_cache, v_cache, block_tables, max_blocks, block_size, seq_lens, cu_q, nullptr, 0, nullptr, window,
-                               nullptr, 0, out, B, max_q, hq, hkv, dk, dv, scale, dtype, stream, nullptr, maps, keep_first, cap, ldo, out_f32);
+  return llmss_attention_span_ex(q, ldq, k_cache, v_cache, dv, block_tables, max_blocks, block_size, seq_lens, cu_q, window, 0, keep_first,
+                                 cap, maps, nullptr, out, ldo, out_f32, B, max_q, hq, hkv, dk, dv, scale, dtype, stream);
 }
 
 // x [T][hq][2][dv] 32-bit -> out [T][hq * dv] (row stride ldo): rms_div(x1 - lam * x2) * factor per head

@@ -17,9 +17,10 @@
 // partially filled page still enter the PV MMA multiplied by P = 0, so cache pages must hold finite values
 // (0 * NaN = NaN).  The engine zero-initialises the pool and pages only ever hold real K/V, so this holds.
 //
-// Span form (llmss_attn_decode_span): a sliding window -- only the key tiles it reaches, and those of the sequence's kept first
-// tokens, are walked --, soft-capped scores, key and value sizes that are any multiple of 8 (the tile is the next of 64 / 128 /
-// 256, columns beyond the size arrive as TMA's zero fill), and two query / key maps per head: the key row holds both maps, the
+// Span form (llmss_attn_decode_span): a sliding window or a chunked mask -- only the key tiles it reaches, and those of the
+// sequence's kept first tokens, are walked --, soft-capped scores, an attention sink per head, values that are the leading columns of
+// wider rows (latent attention), key and value sizes that are any multiple of 8 (the tile is the next of 64 / 128 / 256, columns
+// beyond the size arrive as TMA's zero fill), and two query / key maps per head: the key row holds both maps, the
 // query rows come zero-padded to that width, so a group's 2 G rows share one read of K and V; the combine pass subtracts.
 //
 // Replaces SURVEY.md G8 (`baddbmm` + TorchScript softmax + `bmm` on a replicated KV tensor,
@@ -52,7 +53,7 @@ struct DArgs {
   int q_copies;      // TMA ops per chunk: the same rows land at q_copies row offsets (physical replication)
   int q_alloc_rows;  // rows of one Q buffer in shared memory
   int q_sbo;         // stride between 8-row groups in the Q descriptors (0: every group re-reads rows 0..7)
-  int ws;            // G <= 8, 64-token pages, 64-key tiles: weight-stationary 32-row MMAs (tcgen05.mma.ws), whose
+  int ws;            // G <= 32, 64-token pages, 64-key tiles: weight-stationary 32-row MMAs (tcgen05.mma.ws), whose
                      // accumulator layout puts key / head-dim columns [q*N/4, (q+1)*N/4) into sub-partition q
   int block_size;
   int num_splits;
@@ -72,6 +73,7 @@ struct DArgs {
   int k_ops, v_ops;    // TMA ops per page: 1, or one per 64-column chunk where the size is no multiple of 64
   int k_tx, v_tx;      // bytes per key tile
   int window, keep;    // span form: window 0: none; keys < keep are never hidden
+  int chunk;           // 0: none, else only keys of the last token's own block of `chunk` positions
   float cap_in, cap_log2;   // soft cap: cap_in = scale / cap (0: none), cap_log2 = cap * log2 e
   int partials;        // 1: write partials even when an item covers its whole sequence (the combine pass has more to do)
 };
@@ -80,6 +82,7 @@ struct Item {
   int b, kvh, L, n_tiles;
   int v_begin;          // first tile of this unit in the walk: tiles 0 .. n_first - 1, then t_first .. (see key_tile)
   int t_first, n_first;
+  int lo;       // first visible key (span form)
   int direct;   // this unit covers the whole sequence: write the normalised output, no partial
   int part;     // partial slot within the (sequence, head) row
   int pstride;  // slots per (sequence, head)
@@ -108,7 +111,8 @@ __device__ __forceinline__ Item decode_item(const DArgs& a, int it) {
   r.kvh = t % a.hkv;
   r.b = t / a.hkv;
   r.L = a.seq_lens[r.b];
-  r.t_first = SPAN && a.window > 0 ? max(0, r.L - a.window) / BN : 0;
+  r.lo = SPAN && r.L > 0 ? first_visible(r.L - 1, a.window, a.chunk) : 0;
+  r.t_first = r.lo / BN;
   r.n_first = SPAN ? min((a.keep + BN - 1) / BN, r.t_first) : 0;
   const int total = r.L > 0 ? (r.L + BN - 1) / BN - r.t_first + r.n_first : 0;
   const int chunk = (total + a.num_splits - 1) / a.num_splits;  // whole key tiles per split
@@ -169,7 +173,7 @@ struct Sched {
     r.kvh = kvh;
     r.L = a.seq_lens[b];
     r.v_begin = j;
-    r.t_first = r.n_first = 0;
+    r.t_first = r.n_first = r.lo = 0;
     r.n_tiles = take;
     r.direct = take == n;
     r.part = (int)blockIdx.x - (t - j) / quota;  // CTAs that share this item are consecutive
@@ -557,8 +561,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
           for (int i = 0; i < CW; ++i)
             if (kbase + i >= I.L) sc[i] = -INFINITY;
         }
-        if (SPAN && a.window > 0 && kbase < I.L - a.window && kbase + CW > a.keep) {   // the window starts inside or behind these keys
-          const int lo = I.L - a.window - kbase, kp = a.keep - kbase;
+        if (SPAN && kbase < I.lo && kbase + CW > a.keep) {   // the first visible key lies inside or behind these keys
+          const int lo = I.lo - kbase, kp = a.keep - kbase;
 #pragma unroll
           for (int i = 0; i < CW; ++i)
             if (i < lo && i >= kp) sc[i] = -INFINITY;
@@ -735,7 +739,8 @@ __global__ void attn_decode_tc_balanced_combine_kernel(const float* __restrict__
 template <typename T>
 __global__ void __launch_bounds__(128) attn_decode_span_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                                        T* __restrict__ out, int64_t ldo, int hq, int maps, int D, int dv,
-                                                                       int num_splits, float lam, float eps, float factor) {
+                                                                       int num_splits, float lam, float eps, float factor,
+                                                                       const float* __restrict__ sinks) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[4];
@@ -756,6 +761,7 @@ __global__ void __launch_bounds__(128) attn_decode_span_combine_kernel(const flo
         if (c < dv) at[i] += part_o[(base + s) * D + c] * sc;
       }
     }
+    if (sinks != nullptr && lt > 0.f) lt += exp2f(sinks[head * maps + m] * 1.4426950408889634f - mn);
     const float w = lt > 0.f ? (m == 0 ? 1.f : -lam) / lt : 0.f;
 #pragma unroll
     for (int i = 0; i < 2; ++i) o[i] = fmaf(at[i], w, o[i]);
@@ -863,13 +869,19 @@ LLMSS_API int llmss_attn_decode_tc_pick_splits(int B, int hkv, int d, int max_kv
   return best;
 }
 
+// Weight-stationary MMAs: one 64-token page per 64-key tile and at most 32 query rows (LLMSS_ATTN_WS=0 keeps the other form)
+static bool ws_form(int G, int block_size, int d) {
+  const char* e = getenv("LLMSS_ATTN_WS");
+  return !(e != nullptr && e[0] == '0') && G <= 32 && block_size == 64 && tile_keys(d) == 64;
+}
+
 // Whether llmss_attn_decode_tc can take this head grouping and head size (its query tile and at least two key stages must
 // fit into shared memory): callers with an alternative kernel ask first instead of catching the refusal.
 LLMSS_API int llmss_attn_decode_tc_supported(int hq, int hkv, int d, int block_size) {
   if (!(d == 64 || d == 128 || d == 256) || hq <= 0 || hkv <= 0 || hq % hkv != 0 || hq / hkv > 128) return 0;
   if (!(block_size == 16 || block_size == 32 || block_size == 64)) return 0;
   const int G = hq / hkv;
-  const int q_alloc_rows = G <= 8 ? 8 : (G <= 64 ? 128 : (G + 7) / 8 * 8);
+  const int q_alloc_rows = G <= 8 ? 8 : (G <= 32 && ws_form(G, block_size, d) ? 32 : (G <= 64 ? 128 : (G + 7) / 8 * 8));
   int smem = 0;
   return plan_stages(q_alloc_rows, d, &smem) >= 2 ? 1 : 0;
 }
@@ -881,6 +893,7 @@ struct SpanArgs {
   int dk, dv, maps;      // key row and value size; query / key maps per head (hq counts heads x maps)
   int window, keep;
   float cap, lam, eps, factor;
+  int chunk, ldv;        // chunked mask (0: none); row stride of the V pages
 };
 
 static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
@@ -903,7 +916,9 @@ static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const
   const int G = hq / hkv;
   // Row replication plan (see the kernel comment): R copies of the group's heads down the 128 MMA rows.
   int R, q_box_rows, q_copies, q_alloc_rows, q_sbo;
-  if (G <= 8) { R = 4; q_box_rows = 8; q_copies = 1; q_alloc_rows = 8; q_sbo = 0; }
+  const bool ws = ws_form(G, block_size, d);
+  if (ws && G > 8) { R = 4; q_box_rows = 32; q_copies = 1; q_alloc_rows = 32; q_sbo = 1024; }   // 32 rows, no copies: see umma_f16_ss_ws
+  else if (G <= 8) { R = 4; q_box_rows = 8; q_copies = 1; q_alloc_rows = 8; q_sbo = 0; }
   else if (G <= 32) { R = 4; q_box_rows = 32; q_copies = 4; q_alloc_rows = 128; q_sbo = 1024; }
   else if (G <= 64) { R = 2; q_box_rows = 64; q_copies = 2; q_alloc_rows = 128; q_sbo = 1024; }
   else { R = 1; q_box_rows = (G + 7) / 8 * 8; q_copies = 1; q_alloc_rows = q_box_rows; q_sbo = 1024; }
@@ -928,11 +943,11 @@ static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const
     // landing in shared memory chunk-major ([chunk][block_size rows][128 B]), which is what the MMA
     // descriptors of a page expect -- a single TMA op per page whatever the head size.  A size that is no multiple of 64 goes
     // chunk by chunk instead, so that the columns beyond it are out of the map's range and read as zeros.
-    const int w = which == 0 ? dk : dv;
+    const int w = which == 0 ? dk : dv, ld = which == 0 || span == nullptr ? w : span->ldv;
     const bool whole = w % 64 == 0;
     const cuuint64_t rows = (cuuint64_t)num_blocks * hkv * block_size;
     cuuint64_t dims[3] = {(cuuint64_t)(whole ? 64 : w), rows, (cuuint64_t)(whole ? w / 64 : 1)};
-    cuuint64_t strides[2] = {(cuuint64_t)w * 2, whole ? 128 : rows * w * 2};
+    cuuint64_t strides[2] = {(cuuint64_t)ld * 2, whole ? 128 : rows * ld * 2};
     cuuint32_t box[3] = {64, (cuuint32_t)block_size, (cuuint32_t)(whole ? w / 64 : 1)};
     cuuint32_t estr[3] = {1, 1, 1};
     CUresult r = enc(which == 0 ? &tk : &tv, dt, 3, const_cast<void*>(which == 0 ? k_cache : v_cache), dims, strides, box,
@@ -960,10 +975,7 @@ static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const
   a.q_copies = q_copies;
   a.q_alloc_rows = q_alloc_rows;
   a.q_sbo = q_sbo;
-  {
-    const char* e = getenv("LLMSS_ATTN_WS");  // LLMSS_ATTN_WS=0 falls back to the 64-row tcgen05.mma form
-    a.ws = (!(e != nullptr && e[0] == '0') && G <= 8 && block_size == 64 && tile_keys(d) == 64) ? 1 : 0;
-  }
+  a.ws = ws ? 1 : 0;
   a.block_size = block_size;
   a.num_splits = num_splits;
   a.n_items = B * hkv * num_splits;
@@ -981,6 +993,7 @@ static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const
   a.v_tx = (dv + 63) / 64 * 128 * tile_keys(d);
   if (span != nullptr) {
     a.window = span->window < (1 << 30) ? span->window : 0;
+    a.chunk = span->chunk < (1 << 30) ? span->chunk : 0;
     a.keep = span->keep < (1 << 30) ? span->keep : (1 << 30);
     a.cap_in = span->cap > 0.f ? scale / span->cap : 0.f;
     a.cap_log2 = span->cap * 1.4426950408889634f;
@@ -1012,11 +1025,11 @@ static int decode_tc_impl(const void* q, int64_t ldq, const void* k_cache, const
     const dim3 cgrid(hq / span->maps, B);
     if (dtype == LLMSS_F16)
       LLMSS_CHECK_CUDA(launch_pdl(attn_decode_span_combine_kernel<__half>, cgrid, dim3(128), 0, stream, (const float*)a.part_o, (const float*)a.part_ml,
-                                  (__half*)out, ldo, hq, span->maps, d, dv, num_splits, span->lam, span->eps, span->factor));
+                                  (__half*)out, ldo, hq, span->maps, d, dv, num_splits, span->lam, span->eps, span->factor, a.sinks));
     else
       LLMSS_CHECK_CUDA(launch_pdl(attn_decode_span_combine_kernel<__nv_bfloat16>, cgrid, dim3(128), 0, stream, (const float*)a.part_o,
                                   (const float*)a.part_ml, (__nv_bfloat16*)out, ldo, hq, span->maps, d, dv, num_splits, span->lam, span->eps,
-                                  span->factor));
+                                  span->factor, a.sinks));
     return 0;
   }
   if (balanced) {
@@ -1070,18 +1083,31 @@ LLMSS_API int llmss_attn_decode_tc_sink(const void* q, int64_t ldq, const void* 
 // Span form (one query token per sequence): see the head of the file.  q [B][hq * maps][maps * dk] -- for maps = 2 every row zero
 // outside its own map's columns --, K pages [num_blocks][hkv][block_size][maps * dk], V pages [..][dv], out [B][hq * dv] (row
 // stride ldo).  scratch: llmss_attn_decode_scratch_floats(B, hq * maps, D, num_splits) floats, D = 64 / 128 / 256 the smallest
-// that holds maps * dk and dv; needed for num_splits > 1 or maps = 2.  num_splits >= 1.
-LLMSS_API int llmss_attn_decode_span(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
-                                     int max_blocks, const int* seq_lens, void* out, int64_t ldo, float* scratch, int B, int hq, int hkv,
-                                     int dk, int dv, int maps, int block_size, int num_blocks, float scale, int window, int keep_first,
-                                     float cap, float lam, float eps, float factor, int num_splits, int dtype, cudaStream_t stream) {
+// that holds maps * dk and dv; needed for num_splits > 1 or maps = 2.  num_splits >= 1.  chunk, sinks, ldv: see
+// llmss_attn_prefill_span_ex.
+LLMSS_API int llmss_attn_decode_span_ex(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, int ldv,
+                                        const int* block_tables, int max_blocks, const int* seq_lens, void* out, int64_t ldo,
+                                        float* scratch, int B, int hq, int hkv, int dk, int dv, int maps, int block_size, int num_blocks,
+                                        float scale, int window, int chunk, int keep_first, float cap, const float* sinks, float lam,
+                                        float eps, float factor, int num_splits, int dtype, cudaStream_t stream) {
+  LLMSS_REQUIRE(chunk >= 0 && ldv >= dv && ldv % 8 == 0 && (sinks == nullptr || maps == 1),
+                "attn_decode_span: chunk %d, value rows of %d for %d columns", chunk, ldv, dv);
   LLMSS_REQUIRE(maps == 1 || maps == 2, "attn_decode_span: %d maps", maps);
   LLMSS_REQUIRE(dk > 0 && dv > 0 && dk % 8 == 0 && dv % 8 == 0 && maps * dk <= 256 && dv <= 256,
                 "attn_decode_span: key size %d x %d / value size %d unsupported", maps, dk, dv);
   LLMSS_REQUIRE(scale > 0.f && window >= 0 && keep_first >= 0 && cap >= 0.f && num_splits >= 1, "attn_decode_span: bad scale, window, cap or splits");
   LLMSS_REQUIRE((((uintptr_t)out | (uintptr_t)k_cache | (uintptr_t)v_cache) % 16) == 0, "attn_decode_span: out / pages must be 16-byte aligned");
   const int w = maps * dk > dv ? maps * dk : dv, d = w <= 64 ? 64 : (w <= 128 ? 128 : 256);
-  const SpanArgs sp{maps * dk, dv, maps, window, keep_first, cap, lam, eps, factor};
+  const SpanArgs sp{maps * dk, dv, maps, window, keep_first, cap, lam, eps, factor, chunk, ldv};
   return decode_tc_impl(q, ldq, k_cache, v_cache, block_tables, max_blocks, seq_lens, out, ldo, scratch, B, hq * maps, hkv, d, block_size,
-                        num_blocks, scale, num_splits, dtype, nullptr, 0, stream, nullptr, &sp);
+                        num_blocks, scale, num_splits, dtype, nullptr, 0, stream, sinks, &sp);
+}
+
+LLMSS_API int llmss_attn_decode_span(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
+                                     int max_blocks, const int* seq_lens, void* out, int64_t ldo, float* scratch, int B, int hq, int hkv,
+                                     int dk, int dv, int maps, int block_size, int num_blocks, float scale, int window, int keep_first,
+                                     float cap, float lam, float eps, float factor, int num_splits, int dtype, cudaStream_t stream) {
+  return llmss_attn_decode_span_ex(q, ldq, k_cache, v_cache, dv, block_tables, max_blocks, seq_lens, out, ldo, scratch, B, hq, hkv, dk, dv,
+                                   maps, block_size, num_blocks, scale, window, 0, keep_first, cap, nullptr, lam, eps, factor, num_splits,
+                                   dtype, stream);
 }

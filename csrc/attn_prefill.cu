@@ -20,9 +20,9 @@
 //   the GEMM output in place; `out` may alias q (the fused GPT-J block writes the context over q).
 //   GQA/MQA: kv head = q head / (hq / hkv).
 //
-// Span form (MAPS = 1 / 2, over the paged cache): a sliding window whose hidden key tiles are skipped and that may keep the
-// sequence's first tokens (their tiles come first in the walk), soft-capped scores, and any key / value size that is a
-// multiple of 8 (the tile is the next of 64 / 128 / 256; TMA fills the columns beyond the size with zeros).  MAPS = 2 is
+// Span form (MAPS = 1 / 2, over the paged cache): a sliding window or a chunked mask whose hidden key tiles are skipped and that
+// may keep the sequence's first tokens (their tiles come first in the walk), soft-capped scores, an attention sink per head,
+// values that are the leading columns of wider rows (latent attention), and any key / value size that is a multiple of 8 (the tile is the next of 64 / 128 / 256; TMA fills the columns beyond the size with zeros).  MAPS = 2 is
 // differential attention: a head has two query / key vectors over one value and the key row holds both side by side.  A CTA
 // takes 64 queries; rows 0-63 of its query tile are map 1 and rows 64-127 map 2, each zero outside its own half of the key
 // row (again TMA's fill: the box starts at a shifted column), so ONE MMA per tile forms the scores of both maps from one
@@ -98,6 +98,7 @@ struct PArgs {
   const float* sinks;
   // span form only
   int window, keep;          // window 0: none
+  int chunk;                 // 0: none, else only keys of the query's own block of `chunk` positions
   int dk, dkp, dv;           // one map's key size, the key row's (maps * dk), value size
   float cap_in, cap_log2;    // cap_in > 0: score -> cap * tanh(raw * scale / cap): cap_in = scale / cap, cap_log2 = cap * log2 e
   float lam, eps, factor;    // two maps: rms_div(a1 - lam * a2) * factor
@@ -227,10 +228,8 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
   // window: the walk takes tiles 0 .. n_first - 1 (kept first tokens), then t_first .. (the first row's window on)
   int t_first = 0, n_first = 0;
   if constexpr (SPAN) {
-    if (a.window > 0) {
-      t_first = max(0, ctx + q0 - a.window + 1) / BN;
-      n_first = min((a.keep + BN - 1) / BN, t_first);
-    }
+    t_first = first_visible(ctx + q0, a.window, a.chunk) / BN;
+    n_first = min((a.keep + BN - 1) / BN, t_first);
   }
   const int n_tiles = (kv_end + BN - 1) / BN - t_first + n_first;
   auto key_tile = [&](int j) { return SPAN ? (j < n_first ? j : j - n_first + t_first) : j; };
@@ -413,6 +412,9 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
     const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
     float m_run = -INFINITY, l_run = 0.f;
     const float scale_log2 = (SPAN && a.cap_in > 0.f) ? a.cap_log2 : a.scale_log2;
+    // first visible key of this thread's row, and of the CTA's last row (no tile from there on hides a key below a row's first)
+    const int row_lo = SPAN ? first_visible(qpos, a.window, a.chunk) : 0;
+    const int last_lo = SPAN ? first_visible(ctx + q0 + QT - 1, a.window, a.chunk) : 0;
     for (int j = 0; j < n_tiles; ++j) {
       mbar_wait(&bar_s[j & 1], (j >> 1) & 1, 70);
       tcgen05_fence_after();
@@ -448,10 +450,10 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
       }
       if constexpr (SPAN) {
         if (a.cap_in > 0.f) softcap_scores<BN>(sc, a.cap_in);
-        // some row's window starts inside or behind this tile, and not all of the tile is kept
-        const bool low = a.window > 0 && kbase < ctx + q0 + QT - a.window && kbase + BN > a.keep;
+        // some row's first key lies inside or behind this tile, and not all of the tile is kept
+        const bool low = kbase < last_lo && kbase + BN > a.keep;
         if (diag || low) {
-          const int hi = qpos - kbase, lo = a.window > 0 ? hi - a.window + 1 : -1, kp = a.keep - kbase;
+          const int hi = qpos - kbase, lo = row_lo - kbase, kp = a.keep - kbase;
 #pragma unroll
           for (int i = 0; i < BN; ++i)
             if (i > hi || (i < lo && i >= kp)) sc[i] = -INFINITY;
@@ -541,7 +543,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_const
     // epilogue: O / l -> out
     mbar_wait(&bar_o[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, 72);
     tcgen05_fence_after();
-    if constexpr (BIAS) {
+    if constexpr (BIAS || SPAN) {
       if (a.sinks != nullptr && l_run > 0.f) l_run += exp2f(a.sinks[head] * 1.4426950408889634f - m_run);
     }
     float inv_l = l_run > 0.f ? 1.0f / l_run : 0.f;
@@ -660,7 +662,7 @@ int launch_span(const CUtensorMap& tm, const CUtensorMap& tk, const CUtensorMap&
   return 0;
 }
 
-int encode_2d(CUtensorMap* tm, const void* base, int dtype, int64_t cols, int64_t rows, int64_t ld, int box_rows) {
+int encode_2d(CUtensorMap* tm, const void* base, int dtype, int64_t cols, int64_t rows, int64_t ld, int box_rows) {   // columns beyond `cols` read as zeros
   PFN_encodeTiled enc = get_encode();
   LLMSS_REQUIRE(enc != nullptr, "attn_prefill: cuTensorMapEncodeTiled entry point not available");
   cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
@@ -833,12 +835,15 @@ LLMSS_API int llmss_attn_prefill_paged_sink(const void* q, int64_t ldq, const vo
 // soft-capped scores (cap 0: none) and maps = 1 / 2 query / key vectors per head.  q [total_q][hq * maps][dk] (row stride ldq),
 // K pages [num_blocks][hkv][block_size][maps * dk], V pages [num_blocks][hkv][block_size][dv].  maps = 1: out [total_q][hq * dv]
 // (row stride ldo) holds the attention outputs; maps = 2: rms_div(a1 - lam * a2) * factor per head.  dk and dv multiples of 8,
-// maps * dk and dv at most 256.
-LLMSS_API int llmss_attn_prefill_span(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
-                                      int max_blocks, const int* seq_lens, void* out, int64_t ldo, const int* cu_q, int num_seqs,
-                                      int max_q, int total_q, int hq, int hkv, int dk, int dv, int maps, int block_size, int num_blocks,
-                                      float scale, int window, int keep_first, float cap, float lam, float eps, float factor, int dtype,
-                                      cudaStream_t stream) {
+// maps * dk and dv at most 256.  chunk > 0: only keys of the query's own block of `chunk` positions.  sinks [hq] 32-bit or null (maps =
+// 1): exp(sinks[h]) joins every softmax denominator of head h.  ldv: row stride of the V pages, a multiple of 8 (>= dv).
+LLMSS_API int llmss_attn_prefill_span_ex(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, int ldv,
+                                         const int* block_tables, int max_blocks, const int* seq_lens, void* out, int64_t ldo,
+                                         const int* cu_q, int num_seqs, int max_q, int total_q, int hq, int hkv, int dk, int dv, int maps,
+                                         int block_size, int num_blocks, float scale, int window, int chunk, int keep_first, float cap,
+                                         const float* sinks, float lam, float eps, float factor, int dtype, cudaStream_t stream) {
+  LLMSS_REQUIRE(chunk >= 0 && ldv >= dv && ldv % 8 == 0 && (sinks == nullptr || maps == 1),
+                "attn_prefill_span: chunk %d, value rows of %d for %d columns", chunk, ldv, dv);
   LLMSS_REQUIRE(dtype == LLMSS_F16 || dtype == LLMSS_BF16, "attn_prefill_span: dtype must be f16/bf16");
   LLMSS_REQUIRE(maps == 1 || maps == 2, "attn_prefill_span: %d maps", maps);
   LLMSS_REQUIRE(dk > 0 && dv > 0 && dk % 8 == 0 && dv % 8 == 0 && maps * dk <= 256 && dv <= 256,
@@ -864,7 +869,7 @@ LLMSS_API int llmss_attn_prefill_span(const void* q, int64_t ldq, const void* k_
   LLMSS_REQUIRE(r == CUDA_SUCCESS, "attn_prefill_span: q tensor map failed (CUresult %d)", (int)r);
   const int64_t crow = (int64_t)num_blocks * hkv * block_size;
   if (int e = encode_2d(&tk, k_cache, dtype, maps * dk, crow, maps * dk, block_size)) return e;
-  if (int e = encode_2d(&tv, v_cache, dtype, dv, crow, dv, block_size)) return e;
+  if (int e = encode_2d(&tv, v_cache, dtype, dv, crow, ldv, block_size)) return e;
   PArgs a;
   memset(&a, 0, sizeof(a));
   a.cu_seqlens = cu_q;
@@ -876,6 +881,8 @@ LLMSS_API int llmss_attn_prefill_span(const void* q, int64_t ldq, const void* k_
   a.ldo = ldo;
   a.hq = hq;
   a.hkv = hkv;
+  a.chunk = chunk < (1 << 30) ? chunk : 0;
+  a.sinks = sinks;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.dtype = dtype;
   a.window = window < (1 << 30) ? window : 0;
@@ -902,4 +909,14 @@ LLMSS_API int llmss_attn_prefill_span(const void* q, int64_t ldq, const void* k_
     LLMSS_PS(__nv_bfloat16, 256);
   }
 #undef LLMSS_PS
+}
+
+LLMSS_API int llmss_attn_prefill_span(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const int* block_tables,
+                                      int max_blocks, const int* seq_lens, void* out, int64_t ldo, const int* cu_q, int num_seqs,
+                                      int max_q, int total_q, int hq, int hkv, int dk, int dv, int maps, int block_size, int num_blocks,
+                                      float scale, int window, int keep_first, float cap, float lam, float eps, float factor, int dtype,
+                                      cudaStream_t stream) {
+  return llmss_attn_prefill_span_ex(q, ldq, k_cache, v_cache, dv, block_tables, max_blocks, seq_lens, out, ldo, cu_q, num_seqs, max_q,
+                                    total_q, hq, hkv, dk, dv, maps, block_size, num_blocks, scale, window, 0, keep_first, cap, nullptr, lam,
+                                    eps, factor, dtype, stream);
 }

@@ -300,6 +300,18 @@ __device__ __forceinline__ void fmul2(float& d0, float& d1, float a0, float a1, 
       : "=f"(d0), "=f"(d1) : "f"(a0), "f"(a1), "f"(b0), "f"(b1));
 }
 
+// ---------------------------------------------------------------- visible keys
+// first key position that query position p sees through a sliding window (0: none) and / or a chunked mask (0: none; p sees its own
+// block of `chunk` positions, counted from the sequence's start)
+__host__ __device__ __forceinline__ int first_visible(int p, int window, int chunk) {
+  int lo = window > 0 && p - window + 1 > 0 ? p - window + 1 : 0;
+  if (chunk > 0) {
+    const int c = p - p % chunk;
+    lo = c > lo ? c : lo;
+  }
+  return lo;
+}
+
 // ---------------------------------------------------------------- soft cap
 // tanh for soft-capped attention scores, 32-bit.  |x| <= 0.5: an odd polynomial of degree 9 fitted on that range (relative error
 // 1.1e-7 in 32-bit arithmetic, FMA pipe only); larger: 1 - 2 / (e^(2x) + 1) (absolute error of a few units in the last place of

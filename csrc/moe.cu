@@ -191,7 +191,7 @@ __global__ void __launch_bounds__(256) moe_up_kernel(const T* __restrict__ h, in
 template <typename T>
 __global__ void __launch_bounds__(256) moe_down_kernel(const T* __restrict__ act_in, const int* __restrict__ ids,
                                                        const float* __restrict__ wts, const T* __restrict__ w_down, int64_t ldd,
-                                                       float* __restrict__ out, int64_t ldo, int W, int F, int top) {
+                                                       float* __restrict__ out, int64_t ldo, int W, int F, int top, int add) {
   extern __shared__ float as[];   // [top][F]
   const int64_t t = blockIdx.x;
   for (int c = threadIdx.x; c < top * F; c += 256) as[c] = to_f32(act_in[t * top * F + c]);
@@ -207,7 +207,7 @@ __global__ void __launch_bounds__(256) moe_down_kernel(const T* __restrict__ act
     for (int c = lane; c < F; c += 32) s = fmaf(to_f32(wr[c]), as[k * F + c], s);
     y += wts[t * top + k] * warp_sum(s);
   }
-  if (lane == 0) out[t * ldo + n] = y;
+  if (lane == 0) out[t * ldo + n] = add ? out[t * ldo + n] + y : y;
 }
 
 // a[t, e * F + f] *= dense[t, e]   (dense form: weight each expert's block before the shared down projection)
@@ -219,6 +219,28 @@ __global__ void __launch_bounds__(256) moe_scale_kernel(T* __restrict__ a, int64
     const float w = dense[t * E + c / F];
     a[t * lda + c] = from_f32<T>(to_f32(a[t * lda + c]) * w);
   }
+}
+
+// the same for 16-bit rows of whole 16-byte pieces (F a multiple of 8): grid (T, pieces / 256), a piece per thread; the pieces of
+// unchosen experts are stored as zeros without being read
+template <typename T>
+__global__ void __launch_bounds__(256) moe_scale_vec_kernel(T* __restrict__ a, int64_t lda, const float* __restrict__ dense, int E, int F) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t t = blockIdx.x;
+  const int c = (blockIdx.y * 256 + threadIdx.x) * 8;
+  if (c >= E * F) return;
+  const float w = dense[t * E + c / F];
+  uint4* p = reinterpret_cast<uint4*>(a + t * lda + c);
+  if (w == 0.f) {
+    *p = make_uint4(0u, 0u, 0u, 0u);
+    return;
+  }
+  float v[8];
+  unpack8<T>(*p, v);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) v[i] *= w;
+  *p = pack8<T>(v);
 }
 
 
@@ -282,25 +304,25 @@ __global__ void __launch_bounds__(256) moe_gather_rows_kernel(const T* __restric
 
 __global__ void __launch_bounds__(256) moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ inv,
                                                           const float* __restrict__ wts, float* __restrict__ out, int64_t ldo,
-                                                          int W, int top) {
+                                                          int W, int top, int add) {
   const int64_t t = blockIdx.x;
   for (int c = threadIdx.x; c < W; c += 256) {
     float v = 0.f;
     for (int k = 0; k < top; ++k) v += wts[t * top + k] * y[(int64_t)inv[t * top + k] * W + c];
-    out[t * ldo + c] = v;
+    out[t * ldo + c] = add ? out[t * ldo + c] + v : v;
   }
 }
 
 template <typename T>
 int launch_experts(const void* h, int64_t ldh, const int* ids, const float* wts, const void* w_up, const void* w_down,
-                   int64_t ldd, void* act_scratch, float* out, int64_t ldo, int T_, int W, int F, int top, int act, int gated,
+                   int64_t ldd, void* act_scratch, float* out, int64_t ldo, int T_, int W, int F, int top, int act, int gated, int add,
                    cudaStream_t stream) {
   const size_t sm_up = (size_t)W * 4, sm_dn = (size_t)top * F * 4;
   static PerDeviceSmem g1, g2;
   LLMSS_CHECK_CUDA(g1.ensure(moe_up_kernel<T>, (int)sm_up));
   LLMSS_CHECK_CUDA(g2.ensure(moe_down_kernel<T>, (int)sm_dn));
   moe_up_kernel<T><<<dim3(T_, top, (F + 7) / 8), 256, sm_up, stream>>>((const T*)h, ldh, ids, (const T*)w_up, (T*)act_scratch, W, F, top, act, gated);
-  moe_down_kernel<T><<<dim3(T_, (W + 7) / 8), 256, sm_dn, stream>>>((const T*)act_scratch, ids, wts, (const T*)w_down, ldd, out, ldo, W, F, top);
+  moe_down_kernel<T><<<dim3(T_, (W + 7) / 8), 256, sm_dn, stream>>>((const T*)act_scratch, ids, wts, (const T*)w_down, ldd, out, ldo, W, F, top, add);
   LLMSS_CHECK_CUDA(cudaGetLastError());
   return 0;
 }
@@ -328,17 +350,31 @@ LLMSS_API int llmss_moe_route(const float* z, int64_t ldz, int T_, int E, int to
   return llmss_moe_route_ex(z, ldz, T_, E, top, groups, keep, route_scale, 0, nullptr, 1, 1, ids, wts, dense, stream);
 }
 
-LLMSS_API int llmss_moe_experts(const void* h, int64_t ldh, const int* ids, const float* wts, const void* w_up,
-                                const void* w_down, int64_t ldd, void* act_scratch, float* out, int64_t ldo, int T_, int W, int F, int top,
-                                int act, int gated, int dtype, cudaStream_t stream) {
+// add = 1: the weighted sum of the chosen experts is added to out, else it replaces it
+LLMSS_API int llmss_moe_experts_ex(const void* h, int64_t ldh, const int* ids, const float* wts, const void* w_up,
+                                   const void* w_down, int64_t ldd, void* act_scratch, float* out, int64_t ldo, int T_, int W, int F,
+                                   int top, int act, int gated, int add, int dtype, cudaStream_t stream) {
   LLMSS_REQUIRE(T_ <= 0x7fffffff / 1 && top <= 65535 && (F + 7) / 8 <= 65535 && (W + 7) / 8 <= 65535, "moe_experts: grid too large");
   LLMSS_REQUIRE((size_t)W * 4 <= 200 * 1024 && (size_t)top * F * 4 <= 200 * 1024, "moe_experts: width %d / top * ff %d exceed shared memory", W, top * F);
   if (T_ == 0) return 0;
-  LLMSS_BY_DTYPE(dtype, return (launch_experts<T>(h, ldh, ids, wts, w_up, w_down, ldd, act_scratch, out, ldo, T_, W, F, top, act, gated, stream)));
+  LLMSS_BY_DTYPE(dtype, return (launch_experts<T>(h, ldh, ids, wts, w_up, w_down, ldd, act_scratch, out, ldo, T_, W, F, top, act, gated, add, stream)));
+}
+
+LLMSS_API int llmss_moe_experts(const void* h, int64_t ldh, const int* ids, const float* wts, const void* w_up,
+                                const void* w_down, int64_t ldd, void* act_scratch, float* out, int64_t ldo, int T_, int W, int F, int top,
+                                int act, int gated, int dtype, cudaStream_t stream) {
+  return llmss_moe_experts_ex(h, ldh, ids, wts, w_up, w_down, ldd, act_scratch, out, ldo, T_, W, F, top, act, gated, 0, dtype, stream);
 }
 
 LLMSS_API int llmss_moe_scale(void* a, int64_t lda, const float* dense, int T_, int E, int F, int dtype, cudaStream_t stream) {
   if (T_ == 0) return 0;
+  const int64_t pieces = (int64_t)E * F / 8;
+  if (dtype != LLMSS_F32 && F % 8 == 0 && lda % 8 == 0 && ((uintptr_t)a) % 16 == 0 && (pieces + 255) / 256 <= 65535) {
+    const dim3 grid(T_, (unsigned)((pieces + 255) / 256));
+    if (dtype == LLMSS_F16) LLMSS_CHECK_CUDA(launch_pdl(moe_scale_vec_kernel<__half>, grid, dim3(256), 0, stream, (__half*)a, lda, dense, E, F));
+    else LLMSS_CHECK_CUDA(launch_pdl(moe_scale_vec_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (__nv_bfloat16*)a, lda, dense, E, F));
+    return 0;
+  }
   LLMSS_BY_DTYPE(dtype, (moe_scale_kernel<T><<<T_, 256, 0, stream>>>((T*)a, lda, dense, E, F)));
   LLMSS_CHECK_CUDA(cudaGetLastError());
   return 0;
@@ -367,10 +403,16 @@ LLMSS_API int llmss_moe_gather_rows(const void* h, int64_t ldh, const int* perm,
   return 0;
 }
 
-LLMSS_API int llmss_moe_combine(const float* y, const int* inv, const float* wts, float* out, int64_t ldo, int T_, int W, int top,
-                                cudaStream_t stream) {
+// add = 1: added to out, else out is replaced
+LLMSS_API int llmss_moe_combine_ex(const float* y, const int* inv, const float* wts, float* out, int64_t ldo, int T_, int W, int top,
+                                   int add, cudaStream_t stream) {
   if (T_ <= 0) return 0;
-  moe_combine_kernel<<<T_, 256, 0, stream>>>(y, inv, wts, out, ldo, W, top);
+  moe_combine_kernel<<<T_, 256, 0, stream>>>(y, inv, wts, out, ldo, W, top, add);
   LLMSS_CHECK_CUDA(cudaGetLastError());
   return 0;
+}
+
+LLMSS_API int llmss_moe_combine(const float* y, const int* inv, const float* wts, float* out, int64_t ldo, int T_, int W, int top,
+                                cudaStream_t stream) {
+  return llmss_moe_combine_ex(y, inv, wts, out, ldo, T_, W, top, 0, stream);
 }

@@ -102,7 +102,7 @@ __global__ void __launch_bounds__(kThreads) norm_residual_kernel(
 }
 
 // ------------------------------------------------------------------------------------------------ 32-bit residual stream
-// r = resid + y (y null: r = resid) ; h = LayerNorm / RMS norm of r times weight (+ bias), stored as TO.  One CTA per row, the
+// r = resid + mult * y (y null: r = resid) ; h = LayerNorm / RMS norm of r times weight (+ bias), stored as TO.  One CTA per row, the
 // row in registers (VEC = 4: 16-byte accesses; longer rows are read back from `out_r`), two-pass variance, 32-bit throughout.
 struct RnArgs {
   const float* resid; int64_t ldr;
@@ -110,6 +110,7 @@ struct RnArgs {
   const float* w; const float* bias;
   float* out_r; void* out_h;         // [M, W] contiguous; out_r null: r is not stored (y null)
   int W; float eps; int kind;
+  float mult;                        // factor on y
 };
 constexpr int kRnRegs = 4;
 
@@ -137,7 +138,7 @@ __global__ void __launch_bounds__(kThreads) residual_norm_kernel(RnArgs a) {
       float u[VEC];
       rn_load<VEC>(a.y + t * a.ldy + c, u);
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) v[e] += u[e];
+      for (int e = 0; e < VEC; ++e) v[e] = fmaf(a.mult, u[e], v[e]);
     }
     if (a.out_r != nullptr) {
       float* o = a.out_r + t * (int64_t)W + c;
@@ -220,15 +221,22 @@ int residual_norm_launch(const RnArgs& a, int M, bool vec, cudaStream_t stream) 
 
 // The counterpart of llmss_norm_residual over a 32-bit residual stream: resid [M, W] (row stride ldr), y [M, W] or null, weight /
 // bias 32-bit (bias may be null), out_r [M, W] contiguous (null with y null), out_h [M, W] contiguous in out_dtype.
-LLMSS_API int llmss_residual_norm(const float* resid, int64_t ldr, const float* y, int64_t ldy, const float* weight, const float* bias,
-                                  float* out_r, void* out_h, int M, int W, float eps, int kind, int out_dtype, cudaStream_t stream) {
+// mult: factor on y.
+LLMSS_API int llmss_residual_norm_ex(const float* resid, int64_t ldr, const float* y, int64_t ldy, float mult, const float* weight,
+                                     const float* bias, float* out_r, void* out_h, int M, int W, float eps, int kind, int out_dtype,
+                                     cudaStream_t stream) {
   LLMSS_REQUIRE(W > 0 && weight != nullptr && out_h != nullptr && (y == nullptr || out_r != nullptr), "residual_norm: bad arguments");
   LLMSS_REQUIRE(kind == LLMSS_NORM_LAYER || kind == LLMSS_NORM_RMS, "residual_norm: norm kind %d", kind);
   if (M <= 0) return 0;
-  RnArgs a{resid, ldr, y, ldy, weight, bias, out_r, out_h, W, eps, kind};
+  RnArgs a{resid, ldr, y, ldy, weight, bias, out_r, out_h, W, eps, kind, mult};
   const bool vec = W % 4 == 0 && ldr % 4 == 0 && ldy % 4 == 0 &&
                    ((((uintptr_t)resid) | ((uintptr_t)y) | ((uintptr_t)weight) | ((uintptr_t)bias) | ((uintptr_t)out_r) | ((uintptr_t)out_h)) & 15) == 0;
   LLMSS_BY_DTYPE(out_dtype, return (residual_norm_launch<T>(a, M, vec, stream)));
+}
+
+LLMSS_API int llmss_residual_norm(const float* resid, int64_t ldr, const float* y, int64_t ldy, const float* weight, const float* bias,
+                                  float* out_r, void* out_h, int M, int W, float eps, int kind, int out_dtype, cudaStream_t stream) {
+  return llmss_residual_norm_ex(resid, ldr, y, ldy, 1.f, weight, bias, out_r, out_h, M, W, eps, kind, out_dtype, stream);
 }
 
 LLMSS_API int llmss_norm_residual(const void* x, const void* x2, const void* residual_in, void* residual_out,

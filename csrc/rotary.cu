@@ -5,12 +5,14 @@
 //                        pages, the raw key projection to the V pages, the queries out in the compute type.
 //   norm_rope_kv_write : q, k, v of grouped-query attention: optional RMS norm of every query / key vector with a weight shared by
 //                        the heads, rotation, keys and values to their pages; one or several query / key vectors ("maps") per
-//                        head side by side; queries only for a layer that attends over another layer's pages.
+//                        head side by side; queries only for a layer that attends over another layer's pages; values
+//                        optionally mixed with another layer's values of the same token.
 //   latent_rope_prep   : latent attention with a rotated key part, first stage: RMS norm of the query latent (-> GEMM operand),
 //                        RMS norm of the key / value latent and rotation of the shared key part (-> one cache row), sigmoid of
 //                        the gate columns.
 //   latent_query_rope  : second stage: per head, the unrotated query part (-> operand of the absorption) and the rotated part
 //                        (-> its columns of the absorbed-query buffer).
+//   latent_rope_qkv    : both stages at once where the queries are columns of the same projection (no query latent, no gate).
 //   hgrn_gates         : q = silu(q), k = 1 - f, ln f with f = lower + (1 - lower) sigmoid(f_raw).
 //   sandwich_residual  : r = resid + rms_div(y) * w_post; optional store as a layer output and depth-weighted average of the
 //                        outputs so far; h = rms_div(r) * w_next.  One CTA per token.
@@ -129,8 +131,9 @@ __global__ void __launch_bounds__(256) rope_norm_kv_write_kernel(const float* __
 }
 
 // norm_rope_kv_write: block 256, a warp per vector of the token's row (hq * maps queries, hkv * maps keys, hkv values).  Grid
-// (T, S): a decode batch spreads a token's vectors over S blocks, a prompt keeps them in one.  Vector form (interleaved pairs,
-// sizes that are multiples of four): LPV lanes share a vector (16: short ones, two per warp) and hold NV 4-column groups each in
+// (T, S): a decode batch spreads a token's vectors over S blocks, a prompt keeps them in one.  Vector form (sizes that are
+// multiples of four; pairs (2i, 2i + 1), or (i, i + n) with n a multiple of four, whose partner columns are read again through
+// L1): LPV lanes share a vector (16: short ones, two per warp) and hold NV 4-column groups each in
 // registers from the 16-byte load to the store; the next P vectors are loaded before the first is worked on.  NV = 0: element
 // by element, any size.
 struct NrArgs {
@@ -143,6 +146,8 @@ struct NrArgs {
   void* k_cache; void* v_cache; int bs;
   void* q_out;
   int pad;                                // queries as [hq * maps][maps * dk], zero outside the map's own columns
+  const float* v_first; int64_t ldf;      // [T][hkv * dv] or null: values become (1 - v_lam) * v + v_lam * v_first
+  float v_lam;
 };
 constexpr int kNrVec = 4;                 // most 4-column groups per lane: sizes up to 512 in the vector form
 
@@ -233,7 +238,28 @@ __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
             const float4 wv = *reinterpret_cast<const float4*>(w + c);
             v[p][i][0] *= rstd * wv.x; v[p][i][1] *= rstd * wv.y; v[p][i][2] *= rstd * wv.z; v[p][i][3] *= rstd * wv.w;
           }
-          if (map >= 0) {
+          if (map >= 0 && !a.interleaved) {
+            if (c < 2 * a.n) {
+              const bool second = c >= a.n;
+              const int pc = second ? c - a.n : c + a.n, p0 = second ? pc : c;       // partner column, first pair of the group
+              float4 o = *reinterpret_cast<const float4*>(nr_source(a, t, u) + pc);
+              if (w != nullptr) {
+                const float4 wv = *reinterpret_cast<const float4*>(w + pc);
+                o.x *= rstd * wv.x; o.y *= rstd * wv.y; o.z *= rstd * wv.z; o.w *= rstd * wv.w;
+              }
+              const float ov[4] = {o.x, o.y, o.z, o.w};
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const float so = ov[e] * sn[p0 + e];
+                v[p][i][e] = fmaf(v[p][i][e], cs[p0 + e], second ? so : -so);
+              }
+            }
+          } else if (map < 0 && a.v_first != nullptr) {
+            const float4 f = *reinterpret_cast<const float4*>(a.v_first + t * a.ldf + (int64_t)(u - (nu - a.hkv)) * a.dv + c);
+            const float fv[4] = {f.x, f.y, f.z, f.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[p][i][e] = fmaf(1.f - a.v_lam, v[p][i][e], a.v_lam * fv[e]);
+          } else if (map >= 0) {
 #pragma unroll
             for (int e = 0; e < 4; e += 2) {
               const int pr = (c + e) >> 1;
@@ -275,6 +301,8 @@ __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
           const int pr = a.interleaved ? c >> 1 : (second ? c - a.n : c);
           const float o = normed(a.interleaved ? (c ^ 1) : (second ? c - a.n : c + a.n));
           r = second ? fmaf(r, cs[pr], o * sn[pr]) : fmaf(r, cs[pr], -o * sn[pr]);
+        } else if (map < 0 && a.v_first != nullptr) {
+          r = fmaf(1.f - a.v_lam, r, a.v_lam * a.v_first[t * a.ldf + (int64_t)(u - (nu - a.hkv)) * a.dv + c]);
         }
         dst[c] = from_f32<T>(r);
         if (a.pad && u < a.hq * a.maps)
@@ -299,7 +327,7 @@ template <typename T>
 __global__ void __launch_bounds__(256) latent_rope_prep_kernel(const float* __restrict__ y, int64_t ldy, int q_off, int q_rank, int c_off,
                                                                int R, int rot, int g_off, int n_gate, const float* __restrict__ qn_w,
                                                                const float* __restrict__ cn_w, float eps, const double* __restrict__ freq,
-                                                               int n, float mag, const int* __restrict__ positions,
+                                                               int n, float mag, int interleaved, const int* __restrict__ positions,
                                                                const int* __restrict__ slots, T* __restrict__ cache, int width,
                                                                T* __restrict__ cq_out, float* __restrict__ gate) {
   __shared__ float cs[kMaxPairs], sn[kMaxPairs], red[8];
@@ -320,7 +348,7 @@ __global__ void __launch_bounds__(256) latent_rope_prep_kernel(const float* __re
     T* dst = cache + (int64_t)slot * width;
     for (int i = threadIdx.x; i < R; i += 256) dst[i] = from_f32<T>(row[c_off + i] * rstd * cn_w[i]);
     const float* kr = row + c_off + R;
-    for (int c = threadIdx.x; c < rot; c += 256) dst[R + c] = from_f32<T>(rotated(kr, c, n, true, cs, sn));
+    for (int c = threadIdx.x; c < rot; c += 256) dst[R + c] = from_f32<T>(rotated(kr, c, n, interleaved, cs, sn));
     for (int c = R + rot + threadIdx.x; c < width; c += 256) dst[c] = from_f32<T>(0.f);
   }
   for (int i = threadIdx.x; i < n_gate; i += 256) gate[t * n_gate + i] = 1.f / (1.f + expf(-row[g_off + i]));
@@ -330,7 +358,7 @@ __global__ void __launch_bounds__(256) latent_rope_prep_kernel(const float* __re
 template <typename T, typename TA>
 __global__ void __launch_bounds__(256) latent_query_rope_kernel(const float* __restrict__ q, int64_t ldq, int H, int d, int rot, int R,
                                                                 int width, const double* __restrict__ freq, int n, float mag,
-                                                                const int* __restrict__ positions, T* __restrict__ q_nope,
+                                                                int interleaved, const int* __restrict__ positions, T* __restrict__ q_nope,
                                                                 TA* __restrict__ q_abs) {
   __shared__ float cs[kMaxPairs], sn[kMaxPairs];
   const int64_t t = blockIdx.x;
@@ -344,9 +372,101 @@ __global__ void __launch_bounds__(256) latent_query_rope_kernel(const float* __r
   const int tail = width - R;          // rotated part, then zero padding
   for (int i = threadIdx.x; i < H * tail; i += 256) {
     const int h = i / tail, c = i - h * tail;
-    const float v = c < rot ? rotated(row + (int64_t)h * (d + rot) + d, c, n, true, cs, sn) : 0.f;
+    const float v = c < rot ? rotated(row + (int64_t)h * (d + rot) + d, c, n, interleaved, cs, sn) : 0.f;
     q_abs[t * (int64_t)H * width + (int64_t)h * width + R + c] = from_f32<TA>(v);
   }
+}
+
+// latent_rope_qkv: grid (T, S), block 256, a warp per unit of the token: unit 0 is the cache row (norm of the latent, rotation of
+// the shared key part), unit 1 + h the query of head h (unrotated part to the operand of the absorption, rotated part and padding
+// to its columns of the absorbed-query buffer).  VEC = 4: 16-byte accesses (all sizes and offsets multiples of four).
+struct LqArgs {
+  const float* y; int64_t ldy;
+  int q_off, H, d, c_off, R, rot;
+  const float* cn_w; float eps;
+  const double* freq; int n; float mag; int interleaved;
+  const int* positions; const int* slots;
+  void* cache; int width;
+  void* q_nope; void* q_abs;
+};
+
+template <typename T, int VEC>
+__device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC]) {
+  if constexpr (VEC == 4) *reinterpret_cast<Quad<T>*>(p) = Quad<T>{from_f32<T>(v[0]), from_f32<T>(v[1]), from_f32<T>(v[2]), from_f32<T>(v[3])};
+  else p[0] = from_f32<T>(v[0]);
+}
+template <int VEC>
+__device__ __forceinline__ void load_vec(const float* p, float (&v)[VEC]) {
+  if constexpr (VEC == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+  } else v[0] = p[0];
+}
+
+template <typename T, typename TA, int VEC>
+__global__ void __launch_bounds__(256) latent_rope_qkv_kernel(LqArgs a) {
+  __shared__ float cs[kMaxPairs], sn[kMaxPairs];
+  const int64_t t = blockIdx.x;
+  pdl_launch_dependents();
+  token_angles(a.freq, a.n, a.positions[t], a.mag, cs, sn);      // inputs of the step, not of the kernel in front
+  pdl_wait();
+  __syncthreads();
+  const int warp = blockIdx.y * 8 + (threadIdx.x >> 5), warps = gridDim.y * 8, l = (threadIdx.x & 31) * VEC;
+  const float* row = a.y + t * a.ldy;
+  auto rotated_part = [&](const float* x, int c, float (&v)[VEC]) {   // columns c .. of a rotated part, zeros behind it
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] = c + e < a.rot ? rotated(x, c + e, a.n, a.interleaved, cs, sn) : 0.f;
+  };
+  for (int u = warp; u <= a.H; u += warps) {
+    float v[VEC];
+    if (u == 0) {
+      const int slot = a.slots[t];
+      if (slot < 0) continue;
+      const float* x = row + a.c_off;
+      T* dst = reinterpret_cast<T*>(a.cache) + (int64_t)slot * a.width;
+      float ss = 0.f;
+      for (int c = l; c < a.R; c += 32 * VEC) {
+        load_vec<VEC>(x + c, v);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) ss = fmaf(v[e], v[e], ss);
+      }
+      const float rstd = rsqrtf(warp_sum(ss) / (float)a.R + a.eps);
+      for (int c = l; c < a.R; c += 32 * VEC) {
+        float w[VEC];
+        load_vec<VEC>(x + c, v);
+        load_vec<VEC>(a.cn_w + c, w);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] *= rstd * w[e];
+        store_vec<T, VEC>(dst + c, v);
+      }
+      for (int c = l; c < a.width - a.R; c += 32 * VEC) {
+        rotated_part(x + a.R, c, v);
+        store_vec<T, VEC>(dst + a.R + c, v);
+      }
+      continue;
+    }
+    const int h = u - 1;
+    const float* x = row + a.q_off + (int64_t)h * (a.d + a.rot);
+    T* qn = reinterpret_cast<T*>(a.q_nope) + (t * a.H + h) * (int64_t)a.d;
+    TA* qa = reinterpret_cast<TA*>(a.q_abs) + (t * a.H + h) * (int64_t)a.width + a.R;
+    for (int c = l; c < a.d; c += 32 * VEC) {
+      load_vec<VEC>(x + c, v);
+      store_vec<T, VEC>(qn + c, v);
+    }
+    for (int c = l; c < a.width - a.R; c += 32 * VEC) {
+      rotated_part(x + a.d, c, v);
+      store_vec<TA, VEC>(qa + c, v);
+    }
+  }
+}
+
+template <typename T, typename TA>
+int latent_qkv_launch(const LqArgs& a, int T_, bool vec, cudaStream_t stream) {
+  const int rounds = (a.H + 8) / 8;
+  const dim3 grid(T_, T_ >= 1024 ? 1 : (rounds < 64 ? rounds : 64));
+  if (vec) LLMSS_CHECK_CUDA(launch_pdl(latent_rope_qkv_kernel<T, TA, 4>, grid, dim3(256), 0, stream, a));
+  else LLMSS_CHECK_CUDA(launch_pdl(latent_rope_qkv_kernel<T, TA, 1>, grid, dim3(256), 0, stream, a));
+  return 0;
 }
 
 __global__ void __launch_bounds__(256) hgrn_gates_kernel(const float* __restrict__ y, int64_t ldy, int nqk, const float* __restrict__ lower,
@@ -523,20 +643,22 @@ LLMSS_API int llmss_rope_norm_kv_write(const float* qk, int64_t ld, int hq, int 
 
 // qkv [T][hq*maps*dk | hkv*maps*dk | hkv*dv] 32-bit; q_w / k_w [dk] 32-bit or null (no norm); K pages [blocks][hkv][block_size][maps *
 // dk], V pages [blocks][hkv][block_size][dv]; q_out [T][hq*maps][dk], or [T][hq*maps][maps*dk] with zeros outside the map's own
-// columns (pad = 1).  hkv = 0: queries only.
-LLMSS_API int llmss_norm_rope_kv_write(const float* qkv, int64_t ld, int hq, int hkv, int dk, int dv, int maps, const float* q_w,
-                                       const float* k_w, float eps, const double* freq, int n_pairs, float mag, int interleaved,
-                                       const int* positions, const int* slots, void* k_cache, void* v_cache, int block_size, void* q_out,
-                                       int pad, int T_, int dtype, cudaStream_t stream) {
+// columns (pad = 1).  hkv = 0: queries only.  v_first [T][hkv*dv] 32-bit (row stride ldf) or null: the V pages take
+// (1 - v_lam) * v + v_lam * v_first.
+LLMSS_API int llmss_norm_rope_kv_write_ex(const float* qkv, int64_t ld, int hq, int hkv, int dk, int dv, int maps, const float* q_w,
+                                          const float* k_w, float eps, const double* freq, int n_pairs, float mag, int interleaved,
+                                          const int* positions, const int* slots, void* k_cache, void* v_cache, int block_size,
+                                          void* q_out, int pad, const float* v_first, int64_t ldf, float v_lam, int T_, int dtype,
+                                          cudaStream_t stream) {
   LLMSS_REQUIRE(hq > 0 && hkv >= 0 && dk > 0 && maps >= 1 && (hkv == 0 || dv > 0), "norm_rope_kv_write: bad sizes");
   LLMSS_REQUIRE(hkv == 0 || (k_cache != nullptr && v_cache != nullptr && slots != nullptr && block_size > 0), "norm_rope_kv_write: keys without pages");
   LLMSS_REQUIRE(n_pairs >= 0 && n_pairs <= kMaxPairs && 2 * n_pairs <= dk, "norm_rope_kv_write: %d rotated pairs for head size %d (at most %d)",
                 n_pairs, dk, kMaxPairs);
   if (T_ <= 0) return 0;
   NrArgs a{qkv, ld, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, n_pairs, mag, interleaved, positions, slots, k_cache, v_cache,
-           block_size, q_out, pad};
+           block_size, q_out, pad, v_first, ldf, v_lam};
   const int widest = hkv > 0 && dv > dk ? dv : dk;
-  const bool vec = interleaved && dk % 4 == 0 && widest <= 128 * kNrVec && (hkv == 0 || dv % 4 == 0) && ld % 4 == 0 &&
+  const bool vec = (interleaved || n_pairs % 4 == 0) && ldf % 4 == 0 && (((uintptr_t)v_first) & 15) == 0 && dk % 4 == 0 && widest <= 128 * kNrVec && (hkv == 0 || dv % 4 == 0) && ld % 4 == 0 &&
                    ((((uintptr_t)qkv) | ((uintptr_t)q_w) | ((uintptr_t)k_w) | ((uintptr_t)k_cache) | ((uintptr_t)v_cache) | ((uintptr_t)q_out)) & 15) == 0;
   const bool half = dk <= 64 && widest <= 128;                          // 16 lanes per vector
   const int per = half ? 16 : 8;
@@ -553,36 +675,76 @@ LLMSS_API int llmss_norm_rope_kv_write(const float* qkv, int64_t ld, int hq, int
   return 0;
 }
 
-LLMSS_API int llmss_latent_rope_prep(const float* y, int64_t ldy, int q_off, int q_rank, int c_off, int rank, int rot, int g_off,
-                                     int n_gate, const float* qn_w, const float* cn_w, float eps, const double* freq, int n_pairs,
-                                     float mag, const int* positions, const int* slots, void* cache, int width, void* cq_out,
-                                     float* gate, int T_, int dtype, cudaStream_t stream) {
+LLMSS_API int llmss_norm_rope_kv_write(const float* qkv, int64_t ld, int hq, int hkv, int dk, int dv, int maps, const float* q_w,
+                                       const float* k_w, float eps, const double* freq, int n_pairs, float mag, int interleaved,
+                                       const int* positions, const int* slots, void* k_cache, void* v_cache, int block_size, void* q_out,
+                                       int pad, int T_, int dtype, cudaStream_t stream) {
+  return llmss_norm_rope_kv_write_ex(qkv, ld, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, n_pairs, mag, interleaved, positions, slots,
+                                     k_cache, v_cache, block_size, q_out, pad, nullptr, 0, 0.f, T_, dtype, stream);
+}
+
+// interleaved: pairs (2i, 2i + 1), else (i, i + n_pairs)
+LLMSS_API int llmss_latent_rope_prep_ex(const float* y, int64_t ldy, int q_off, int q_rank, int c_off, int rank, int rot, int g_off,
+                                        int n_gate, const float* qn_w, const float* cn_w, float eps, const double* freq, int n_pairs,
+                                        float mag, int interleaved, const int* positions, const int* slots, void* cache, int width,
+                                        void* cq_out, float* gate, int T_, int dtype, cudaStream_t stream) {
   LLMSS_REQUIRE(rank > 0 && rot >= 0 && width >= rank + rot, "latent_rope_prep: cache row %d for rank %d + %d rotated", width, rank, rot);
   LLMSS_REQUIRE(n_pairs >= 0 && n_pairs <= kMaxPairs && 2 * n_pairs <= rot, "latent_rope_prep: %d rotated pairs for %d channels", n_pairs, rot);
   if (T_ <= 0) return 0;
   LLMSS_BY_DTYPE(dtype, (latent_rope_prep_kernel<T><<<T_, 256, 0, stream>>>(y, ldy, q_off, q_rank, c_off, rank, rot, g_off, n_gate, qn_w, cn_w,
-                                                                           eps, freq, n_pairs, mag, positions, slots, (T*)cache, width,
+                                                                           eps, freq, n_pairs, mag, interleaved, positions, slots, (T*)cache, width,
                                                                            (T*)cq_out, gate)));
   LLMSS_CHECK_CUDA(cudaGetLastError());
   return 0;
 }
 
+LLMSS_API int llmss_latent_rope_prep(const float* y, int64_t ldy, int q_off, int q_rank, int c_off, int rank, int rot, int g_off,
+                                     int n_gate, const float* qn_w, const float* cn_w, float eps, const double* freq, int n_pairs,
+                                     float mag, const int* positions, const int* slots, void* cache, int width, void* cq_out,
+                                     float* gate, int T_, int dtype, cudaStream_t stream) {
+  return llmss_latent_rope_prep_ex(y, ldy, q_off, q_rank, c_off, rank, rot, g_off, n_gate, qn_w, cn_w, eps, freq, n_pairs, mag, 1, positions,
+                                   slots, cache, width, cq_out, gate, T_, dtype, stream);
+}
+
 // abs_f32: the absorbed-query buffer is 32-bit (generic attention kernel), else it has the compute type
-LLMSS_API int llmss_latent_query_rope(const float* q, int64_t ldq, int H, int d, int rot, int rank, int width, const double* freq,
-                                      int n_pairs, float mag, const int* positions, void* q_nope, void* q_abs, int abs_f32, int T_,
-                                      int dtype, cudaStream_t stream) {
+LLMSS_API int llmss_latent_query_rope_ex(const float* q, int64_t ldq, int H, int d, int rot, int rank, int width, const double* freq,
+                                         int n_pairs, float mag, int interleaved, const int* positions, void* q_nope, void* q_abs,
+                                         int abs_f32, int T_, int dtype, cudaStream_t stream) {
   LLMSS_REQUIRE(H > 0 && d > 0 && width >= rank + rot, "latent_query_rope: bad sizes");
   LLMSS_REQUIRE(n_pairs >= 0 && n_pairs <= kMaxPairs && 2 * n_pairs <= rot, "latent_query_rope: %d rotated pairs for %d channels", n_pairs, rot);
   if (T_ <= 0) return 0;
   if (abs_f32 || dtype == LLMSS_F32) {
     LLMSS_BY_DTYPE(dtype, (latent_query_rope_kernel<T, float><<<T_, 256, 0, stream>>>(q, ldq, H, d, rot, rank, width, freq, n_pairs, mag,
-                                                                                     positions, (T*)q_nope, (float*)q_abs)));
+                                                                                     interleaved, positions, (T*)q_nope, (float*)q_abs)));
   } else {
     LLMSS_BY_DTYPE(dtype, (latent_query_rope_kernel<T, T><<<T_, 256, 0, stream>>>(q, ldq, H, d, rot, rank, width, freq, n_pairs, mag,
-                                                                                 positions, (T*)q_nope, (T*)q_abs)));
+                                                                                 interleaved, positions, (T*)q_nope, (T*)q_abs)));
   }
   LLMSS_CHECK_CUDA(cudaGetLastError());
   return 0;
+}
+
+LLMSS_API int llmss_latent_query_rope(const float* q, int64_t ldq, int H, int d, int rot, int rank, int width, const double* freq,
+                                      int n_pairs, float mag, const int* positions, void* q_nope, void* q_abs, int abs_f32, int T_,
+                                      int dtype, cudaStream_t stream) {
+  return llmss_latent_query_rope_ex(q, ldq, H, d, rot, rank, width, freq, n_pairs, mag, 1, positions, q_nope, q_abs, abs_f32, T_, dtype, stream);
+}
+
+// y [T][*] 32-bit holds the queries [H * (d + rot)] from column q_off on and [latent (rank) | key part (rot)] from column c_off on;
+// cache rows [slot][width >= rank + rot]; q_nope [T][H * d] in dtype, q_abs [T][H * width] in dtype (32-bit if abs_f32), its columns
+// below rank of every head untouched.
+LLMSS_API int llmss_latent_rope_qkv(const float* y, int64_t ldy, int q_off, int H, int d, int c_off, int rank, int rot, const float* cn_w,
+                                    float eps, const double* freq, int n_pairs, float mag, int interleaved, const int* positions,
+                                    const int* slots, void* cache, int width, void* q_nope, void* q_abs, int abs_f32, int T_, int dtype,
+                                    cudaStream_t stream) {
+  LLMSS_REQUIRE(H > 0 && d > 0 && rank > 0 && rot >= 0 && width >= rank + rot, "latent_rope_qkv: bad sizes");
+  LLMSS_REQUIRE(n_pairs >= 0 && n_pairs <= kMaxPairs && 2 * n_pairs <= rot, "latent_rope_qkv: %d rotated pairs for %d channels", n_pairs, rot);
+  if (T_ <= 0) return 0;
+  const LqArgs a{y, ldy, q_off, H, d, c_off, rank, rot, cn_w, eps, freq, n_pairs, mag, interleaved, positions, slots, cache, width, q_nope, q_abs};
+  const bool vec = (ldy | (int64_t)(q_off | d | c_off | rank | rot | width)) % 4 == 0 &&
+                   ((((uintptr_t)y) | ((uintptr_t)cn_w) | ((uintptr_t)cache) | ((uintptr_t)q_nope) | ((uintptr_t)q_abs)) & 15) == 0;
+  if (abs_f32 || dtype == LLMSS_F32) LLMSS_BY_DTYPE(dtype, return (latent_qkv_launch<T, float>(a, T_, vec, stream)));
+  LLMSS_BY_DTYPE(dtype, return (latent_qkv_launch<T, T>(a, T_, vec, stream)));
 }
 
 LLMSS_API int llmss_hgrn_gates(const float* y, int64_t ldy, int n_qk, const float* lower, float* q, float* k, float* logf, int T_,

@@ -65,29 +65,44 @@ class LatentAttention:
 
 
 class RotaryLatentAttention:
-    """Multi-head attention over a low-rank latent with a query latent and a rotated key part shared by all heads.
+    """Multi-head attention over a low-rank latent with a rotated key part shared by all heads.
 
-        c_q = rmsnorm(W_dq h) * g_q ;  q_h = W_uq,h c_q = [q_h^n (dim) | q_h^r (rot)]
-        [c' | k^r] = W_dkv h ;  c = rmsnorm(c') * g_c  (rank) ;  k^r, q_h^r rotated by position (interleaved pairs, table)
+        c_q = rmsnorm(W_dq h) * g_q ;  q_h = W_uq,h c_q = [q_h^n (dim) | q_h^r (rot)]       (q_rank 0: q_h = W_q,h h)
+        [c' | k^r] = W_dkv h ;  c = rmsnorm(c') * g_c  (rank) ;  k^r, q_h^r rotated by position (table; pairs (2i, 2i + 1) if
+        ``interleaved``, else (i, i + n))
         score_h = scale * (q_h^n . W_uk,h c + q_h^r . k^r) ;  causal softmax ;  o_h = sum_j p_hj W_uv,h c_j
-        out = W_o (concat_h(o_h) * sigmoid(W_g h))            the gate is per channel and reads the layer's input
+        out = W_o (concat_h(o_h) * sigmoid(W_g h))            the gate is per channel and reads the layer's input (``gated``)
+
+    ``span``: the form with a sliding ``window`` (0: none) and a sink logit per head in the softmax denominator (``sinks``, or None).
+    It runs on ops.attention_bias with the cache rows as keys and their first ``rank`` columns as values.
 
     Cached per token: [c | k^r] (rank + rot numbers).  Executed in the absorbed form of ``LatentAttention``: with
     q~_h = [W_uk,h^T q_h^n | q_h^r] the score is scale * q~_h . [c | k^r], so the cache row is key AND value of one shared
     head -- the value product carries rot extra columns that the un-absorption never reads.  ``width`` is the cache
     row: rank + rot, or the next size the tcgen05 multi-query kernels take (64 / 128 / 256, zero padded) where that costs
-    at most a quarter more (16-bit CUDA).  The rotation is given as a frequency table and a magnitude
+    at most a quarter more (16-bit CUDA); the span form keeps rank + rot, rounded up to a multiple of 8.  The rotation is given as a frequency table and a magnitude
     (ops.rotary_frequencies), so any frequency schedule fits."""
 
-    def __init__(self, heads: int, dim: int, rot: int, vdim: int, rank: int, q_rank: int, scale: float, eps: float, freq, mag: float):
+    b_in = b_o = None
+
+    def __init__(self, heads: int, dim: int, rot: int, vdim: int, rank: int, q_rank: int, scale: float, eps: float, freq, mag: float = 1.0,
+                 interleaved: bool = True, gated: bool = True, span: bool = False, window: int = 0):
         self.heads, self.dim, self.rot, self.vdim, self.rank, self.q_rank = heads, dim, rot, vdim, rank, q_rank
-        self.scale, self.eps, self.freq, self.mag = scale, eps, freq, mag
+        self.scale, self.eps, self.freq, self.mag, self.interleaved, self.gated = scale, eps, freq, mag, interleaved, gated
+        self.span, self.window, self.sinks = span, int(window or 0), None
+        assert span or not window
+        assert q_rank > 0 or not gated, "latent attention: the gate belongs to the form with a query latent"
         self.width = rank + rot
+        self.w_in = self.w_q = None          # one input GEMM of its own (finalize); W_q of the form without a query latent
         self.w_dq = self.qn_w = self.w_uq = self.w_dkv = self.cn_w = self.w_uk = self.w_uv = self.w_g = self.w_o = None
         self.q_off = self.c_off = self.g_off = 0
 
     def choose_width(self, device, dtype) -> int:
         need = self.rank + self.rot
+        if self.span:
+            if torch.device(device).type == "cuda" and dtype != torch.float32 and self.rank % 8 == 0:
+                self.width = -(-need // 8) * 8
+            return self.width
         if torch.device(device).type == "cuda" and dtype != torch.float32:
             for w in (64, 128, 256):
                 if need <= w and 4 * (w - need) <= w:
@@ -96,39 +111,73 @@ class RotaryLatentAttention:
         return self.width
 
     def weights(self):
-        return [self.w_dq, self.qn_w, self.w_uq, self.w_dkv, self.cn_w, self.w_uk, self.w_uv, self.w_g, self.w_o]
+        return [self.w_in, self.w_q, self.w_dq, self.qn_w, self.w_uq, self.w_dkv, self.cn_w, self.w_uk, self.w_uv, self.w_g, self.sinks, self.w_o]
+
+    @property
+    def n_out(self) -> int:
+        return self.heads * self.vdim
 
     def in_rows(self):
-        return torch.cat([self.w_dq, self.w_dkv, self.w_g], dim=0)
+        return torch.cat([self.w_dq if self.q_rank > 0 else self.w_q, self.w_dkv] + ([self.w_g] if self.gated else []), dim=0)
+
+    def finalize(self):
+        """The projection rows as one operand of this block's own (a layer may add rows behind them)."""
+        self.w_in = self.in_rows().contiguous()
+        assert self.bind(0) == self.w_in.shape[0]
 
     def bind(self, base: int):
         self.q_off = base
-        self.c_off = base + self.q_rank
+        self.c_off = base + (self.q_rank or self.heads * (self.dim + self.rot))
         self.g_off = self.c_off + self.rank + self.rot
-        self.w_dq = self.w_dkv = self.w_g = None
+        self.w_q = self.w_dq = self.w_dkv = self.w_g = None
         self.freq = self.freq.to(torch.float64).to(self.w_o.device).contiguous()     # the kernels read the table on the device
         H, d, R = self.heads, self.dim, self.rank
         # [(head, dim), rank] -> [(head, rank), dim]: the absorption contracts over dim (see LatentAttention.bind)
         self.w_uk = self.w_uk.view(H, d, R).transpose(1, 2).contiguous().view(H * R, d)
-        return self.g_off + H * self.vdim
+        return self.g_off + (H * self.vdim if self.gated else 0)
 
-    def forward(self, y, batch, cache, dtype):
-        """y: the layer's fused 32-bit projection [T, *]; cache: this layer's latent plane [blocks, block_size, width]."""
+    def context_projected(self, y, batch, cache, dtype, out=None):
+        """The concatenated heads [T, heads * vdim] in front of W_o (into ``out`` if given).  y: the layer's fused 32-bit projection
+        [T, *]; cache: this layer's latent plane [blocks, block_size, width]."""
         H, d, r, R, Wd = self.heads, self.dim, self.rot, self.rank, self.width
-        with trace("latent_prep"):
-            cq, gate = ops.latent_rope_prep(y, self.q_off, self.q_rank, self.c_off, R, r, self.g_off, H * self.vdim, self.qn_w,
-                                            self.cn_w, self.eps, self.freq, self.mag, batch.positions, batch.slot_mapping, cache, dtype)
-        with trace("gemm_uq"):
-            q = ops.linear(cq, self.w_uq, out_dtype=torch.float32)
-        with trace("latent_query_rope"):
-            q_nope, q_abs = ops.latent_query_rope(q, H, d, r, R, Wd, self.freq, self.mag, batch.positions, dtype,
-                                                  ops.latent_query_dtype(cache, H, Wd))
+        abs_dtype = dtype if self.span else ops.latent_query_dtype(cache, H, Wd)
+        gate = None
+        if self.q_rank == 0:
+            with trace("latent_prep"):
+                q_nope, q_abs = ops.latent_rope_qkv(y, self.q_off, H, d, self.c_off, R, r, self.cn_w, self.eps, self.freq, self.mag,
+                                                    self.interleaved, batch.positions, batch.slot_mapping, cache, dtype, abs_dtype)
+        else:
+            with trace("latent_prep"):
+                cq, gate = ops.latent_rope_prep(y, self.q_off, self.q_rank, self.c_off, R, r, self.g_off, H * self.vdim if self.gated else 0,
+                                                self.qn_w, self.cn_w, self.eps, self.freq, self.mag, batch.positions, batch.slot_mapping,
+                                                cache, dtype, self.interleaved)
+            with trace("gemm_uq"):
+                q = ops.linear(cq, self.w_uq, out_dtype=torch.float32)
+            with trace("latent_query_rope"):
+                q_nope, q_abs = ops.latent_query_rope(q, H, d, r, R, Wd, self.freq, self.mag, batch.positions, dtype, abs_dtype,
+                                                      self.interleaved)
         with trace("latent_absorb"):
             ops.heads_matmul(q_nope, self.w_uk, H, d, R, False, out=q_abs, out_head_stride=Wd)
         with trace("latent_attention"):
-            o_lat = ops.latent_attention(q_abs, cache, batch, H, Wd, self.scale, dtype)
+            if self.span:
+                pages = cache.view(cache.shape[0], 1, cache.shape[1], Wd)      # one key / value head: the row is the key, its latent the value
+                o_lat, stride = ops.attention_bias(q_abs, pages, pages[..., :R], batch, H, 1, Wd, R, self.scale, None, out_dtype=dtype,
+                                                   window=self.window, sinks=self.sinks), R
+            else:
+                o_lat, stride = ops.latent_attention(q_abs, cache, batch, H, Wd, self.scale, dtype), Wd
         with trace("latent_unabsorb"):
-            ctx = ops.heads_matmul(o_lat, self.w_uv, H, R, self.vdim, False, elem_scale=gate, x_head_stride=Wd, out_dtype=dtype)
+            return ops.heads_matmul(o_lat, self.w_uv, H, R, self.vdim, False, elem_scale=gate, x_head_stride=stride, out_dtype=dtype, out=out)
+
+    def context(self, h, batch, lc, dtype, out=None, y=None, carry=None):
+        """The mixer interface of mixers.ParallelBlock; ``y``: the 32-bit projection by ``w_in``, if it is there already."""
+        if y is None:
+            with trace("gemm_in"):
+                y = ops.linear(h, self.w_in, out_dtype=torch.float32)
+        return self.context_projected(y, batch, lc.latent, dtype, out)
+
+    def forward(self, y, batch, cache, dtype):
+        """y and cache as for ``context_projected``; returns the block's 32-bit output [T, width]."""
+        ctx = self.context_projected(y, batch, cache, dtype)
         with trace("gemm_out"):
             return ops.linear(ctx, self.w_o, out_dtype=torch.float32)
 
@@ -164,6 +213,7 @@ class RoutedExperts:
         # a group scores as the sum of its ``group_top`` best; weights renormalised over the chosen experts or not
         self.score, self.group_top, self.renorm, self.correction = score, group_top, renorm, None
         self.z_off = 0
+        self.b_router = None                               # [E], or no bias on the router logits
         self.w_router = self.w_up = self.w_down = None     # [E, W] | [E, F or 2 F, W] | [W, E * F]
 
     def in_rows(self):
@@ -187,34 +237,57 @@ class RoutedExperts:
     def _route_kw(self):
         return dict(score=self.score, correction=self.correction, group_top=self.group_top, renorm=self.renorm)
 
-    def forward(self, h, y=None):
-        """``y``: a fused projection that holds the router logits at ``z_off`` (32-bit); without it the router runs as
-        a GEMM of its own (32-bit accumulation and output)."""
-        E, F = self.experts, self.ff
+    @property
+    def n_hidden(self) -> int:
+        """Columns of the dense form's hidden row: every expert's."""
+        return self.experts * self.ff
+
+    def form(self, h) -> str:
+        """Which of the three forms a batch runs: "grouped", "dense" or "gather"."""
+        T = h.shape[0]
+        if h.is_cuda and h.dtype != torch.float32:
+            if (T * self.top >= _GROUPED_ROWS * self.experts and self._grouped_pays(T, h.shape[1])
+                    and not torch.cuda.is_current_stream_capturing()):
+                return "grouped"
+            if T >= (_DENSE_MIN or -(-self.experts // self.top)):
+                return "dense"
+        return "gather"
+
+    def _logits(self, y):
+        return y[:, self.z_off:self.z_off + self.experts]
+
+    def weigh(self, a, y):
+        """Dense form: scale every expert's block of the hidden rows ``a`` [T, E * F] by its routing weight (0 if not chosen)."""
+        from ..ops import cuda_impl as cu
+
+        with trace("experts_route"):
+            _, _, dense = cu.moe_route(self._logits(y), self.experts, self.top, self.groups, self.keep, self.route_scale, dense=True,
+                                       **self._route_kw())
+        with trace("experts_weigh"):
+            cu.moe_scale(a, dense, self.experts, self.ff)
+
+    def forward(self, h, y=None, base=None, form=None):
+        """``y``: a fused projection that holds the router logits at ``z_off`` (32-bit, bias included); without it the router runs as
+        a GEMM of its own (32-bit accumulation and output).  ``base`` [T, W] 32-bit: the result is added to it in place (gather and
+        grouped form)."""
+        E = self.experts
         if y is None:
             with trace("experts_router"):
-                y = ops.linear(h, self.w_router, out_dtype=torch.float32)
-        z = y[:, self.z_off:self.z_off + E]
-        T = h.shape[0]
-        if (h.is_cuda and h.dtype != torch.float32 and T * self.top >= _GROUPED_ROWS * E and self._grouped_pays(T, h.shape[1])
-                and not torch.cuda.is_current_stream_capturing()):
-            from ..ops import cuda_impl as cu
-
-            with trace("experts_route"):
-                ids, wts = ops.moe_route(z, E, self.top, self.groups, self.keep, self.route_scale, **self._route_kw())
-            with trace("experts_grouped"):
-                return cu.moe_experts_grouped(h, ids, wts, self.w_up, self.w_down, self.act, self.gated)
-        if h.is_cuda and h.dtype != torch.float32 and T >= (_DENSE_MIN or -(-E // self.top)):
-            from ..ops import cuda_impl as cu
-
-            with trace("experts_route"):
-                _, _, dense = cu.moe_route(z, E, self.top, self.groups, self.keep, self.route_scale, dense=True, **self._route_kw())
+                y = ops.linear(h, self.w_router, self.b_router, out_dtype=torch.float32)
+        form = form or self.form(h)
+        if form == "dense":
+            assert base is None
             with trace("experts_dense_up"):
                 a = ops.linear(h, self.w_up.view(self.w_up.shape[0] * self.w_up.shape[1], -1), act=self.act, gated=self.gated)
-                cu.moe_scale(a, dense, E, F)
+            self.weigh(a, y)
             with trace("experts_dense_down"):
                 return ops.linear(a, self.w_down, out_dtype=torch.float32)
         with trace("experts_route"):
-            ids, wts = ops.moe_route(z, E, self.top, self.groups, self.keep, self.route_scale, **self._route_kw())
+            ids, wts = ops.moe_route(self._logits(y), E, self.top, self.groups, self.keep, self.route_scale, **self._route_kw())
+        if form == "grouped":
+            from ..ops import cuda_impl as cu
+
+            with trace("experts_grouped"):
+                return cu.moe_experts_grouped(h, ids, wts, self.w_up, self.w_down, self.act, self.gated, base)
         with trace("experts_gather"):
-            return ops.moe_experts(h, ids, wts, self.w_up, self.w_down, self.act, self.gated)
+            return ops.moe_experts(h, ids, wts, self.w_up, self.w_down, self.act, self.gated, base)

@@ -20,6 +20,7 @@ from .bedovik import BedovikLM, bedovik_spec, load_bedovik
 from .botalorn import BotalornLM, botalorn_spec, load_botalorn
 from .decoder import DecoderLM
 from .families import FAMILIES
+from .fipavik import FipavikLM, fipavik_spec, load_fipavik
 from .ninelix import NinelixLM, load_ninelix, ninelix_spec
 from .rofulorn import RofulornLM, load_rofulorn, rofulorn_spec
 from .zenorax import ZenoraxLM, load_zenorax, zenorax_spec
@@ -197,6 +198,21 @@ class RofulornForCausalLM(CausalLM):
         self.core.finalize()
 
 
+class FipavikForCausalLM(CausalLM):
+    """Native architecture (see models/fipavik.py): parallel sub-layers over a 32-bit residual stream, windowed latent attention and
+    chunked attention with sinks, value mixing, routed plus shared experts.  Same constructor and forward interface as the
+    HF-shaped classes."""
+    family = "fipavik"
+    float32_on_cuda = True
+
+    def __init__(self, config, weights, fuse_parallel: bool = True):
+        nn.Module.__init__(self)
+        self.config = config
+        self.core = FipavikLM(fipavik_spec(config), weights.process_group, weights.device, weights.dtype)
+        load_fipavik(self.core, weights)
+        self.core.finalize()
+
+
 MODEL_REGISTRY = {
     "gptj": GPTJForCausalLM,
     "gpt_bigcode": GPTBigCodeForCausalLM,
@@ -208,4 +224,5 @@ MODEL_REGISTRY = {
     "botalorn": BotalornForCausalLM,
     "zenorax": ZenoraxForCausalLM,
     "rofulorn": RofulornForCausalLM,
+    "fipavik": FipavikForCausalLM,
 }

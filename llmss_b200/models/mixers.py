@@ -13,13 +13,15 @@
   * ``SinkAttention`` -- grouped-query softmax attention whose values are the projected keys, with rotary positions from
     a frequency table, unit-RMS queries / keys and a learned sink logit per head in the softmax denominator;
   * ``RotaryAttention`` -- grouped-query softmax attention with rotary positions from a frequency table, an optional query /
-    key norm per head, a sliding window that may keep the first tokens, soft-capped scores, optionally two maps per head that
-    are subtracted (differential attention); a layer may attend over the pages another layer writes;
+    key norm per head, a sliding window or a chunked mask that may keep the first tokens, soft-capped scores, an optional sink per
+    head, optionally two maps per head that are subtracted (differential attention); a layer may attend over the pages another
+    layer writes, or mix its values with those of the first mixing layer;
   * ``Hgrn2Mixer`` -- a gated linear recurrence whose forget gate (bounded from below) also sets the write strength;
   * ``DeltaMixer`` -- the gated delta rule (ops.delta_scan) behind short convolutions, with a gated per-head norm;
   * ``HyperConnection`` -- the read / mix / write weights of one sub-layer over several residual streams;
   * ``DenseFFN``, ``GatedFFN``;
-  * ``ParallelBlock`` -- a mixer and a feed-forward that read the same normed input and are summed, with one output product.
+  * ``ParallelBlock`` -- a mixer, a feed-forward and / or routed experts that read the same normed input and are summed, with one
+    input and one output product.
 
 Every block says what it keeps per sequence (``state_shapes``), which cache pages it needs (``kv_shape``), and maps
 (x: the 32-bit residual, h: x in the compute type) to a 32-bit [T, width] output.  All sizes and constants are
@@ -431,22 +433,26 @@ class RotaryAttention:
 
         q, k, v = W h (+ b)  ->  q, k: per head and map rms_div * weight (if ``set_weights`` got norm weights), then rotation
         s_ij = scale * q_i . k_j ;  s <- softcap * tanh(s / softcap)                              (softcap 0: no cap)
-        i sees j <= i with i - j < window or j < keep_first                                       (window 0: every j <= i)
-        plain:         o_h = softmax(s) v
+        i sees j <= i with i - j < window and i // chunk = j // chunk, or j < keep_first          (0: no such limit)
+        plain:         o_h = softmax(s) v          (with sinks: exp(sink_h) is one more term of the denominator)
         differential:  two maps of size dim per head over one value,  o_h = rms_div(a_1 - lam a_2) * (1 - diff),
                        lam = exp(lq1 . lk1) - exp(lq2 . lk2) + diff                               (one number per layer)
         out = W_o concat_h(o) (+ b)
 
     Cached: normed and rotated keys (both maps of a head in one row of its K page) and the projected values.  ``kv_from`` =
     key of another layer: this layer has no key / value tensors and attends over that layer's pages with its own queries, mask
-    and combination.  One input GEMM over the stacked rows [q | k | v]."""
+    and combination.  ``v_mix``: "first" leaves this layer's projected values in the step's ``carry``, "later" caches
+    (1 - v_lam) v + v_lam v_first of the same tokens (``v_lam``: the layer's own number).  One input GEMM over the stacked rows
+    [q | k | v]."""
 
     def __init__(self, width, heads, kv_heads, dim, vdim, scale, eps, freq, mag=1.0, interleaved=True, window=0, keep_first=0,
-                 softcap=0.0, diff=None, kv_from=None):
+                 softcap=0.0, diff=None, kv_from=None, chunk=0, v_mix=None):
         self.width, self.heads, self.kv_heads, self.dim, self.vdim, self.scale, self.eps = width, heads, kv_heads, dim, vdim, scale, eps
         self.freq, self.mag, self.interleaved = freq, mag, interleaved
         self.window, self.keep_first, self.softcap = int(window or 0), int(keep_first or 0), float(softcap or 0.0)
         self.diff, self.maps, self.kv_from, self.own_kv = diff, (1 if diff is None else 2), kv_from, kv_from is None
+        self.chunk, self.v_mix, self.v_lam, self.sinks = int(chunk or 0), v_mix, 0.0, None
+        assert v_mix in (None, "first", "later") and (v_mix is None or self.own_kv)
         assert heads % kv_heads == 0, "rotary attention: query heads must be a multiple of key/value heads"
         assert 2 * freq.numel() <= dim, "rotary attention: more rotated channels than the head has"
         self.w_in = self.b_in = self.q_norm = self.k_norm = self.w_o = self.b_o = None
@@ -463,10 +469,13 @@ class RotaryAttention:
         return (self.kv_heads, self.maps * self.dim, self.vdim) if self.own_kv else None
 
     def weights(self):
-        return [self.w_in, self.b_in, self.q_norm, self.k_norm, self.w_o, self.b_o]
+        return [self.w_in, self.b_in, self.q_norm, self.k_norm, self.sinks, self.w_o, self.b_o]
 
-    def set_weights(self, wq, wk, wv, w_o, bq=None, bk=None, bv=None, b_o=None, q_norm=None, k_norm=None, lam_vectors=None):
-        """wk / wv / bk / bv / k_norm are None for a layer that borrows its keys and values; ``lam_vectors``: (lq1, lk1, lq2, lk2)."""
+    def set_weights(self, wq, wk, wv, w_o, bq=None, bk=None, bv=None, b_o=None, q_norm=None, k_norm=None, lam_vectors=None, sinks=None,
+                    v_lam=0.0):
+        """wk / wv / bk / bv / k_norm are None for a layer that borrows its keys and values; ``lam_vectors``: (lq1, lk1, lq2, lk2);
+        ``sinks`` [heads] 32-bit; ``v_lam``: share of the first mixing layer's values."""
+        self.sinks, self.v_lam = sinks, float(v_lam)
         ws = [wq, wk, wv] if self.own_kv else [wq]
         bs = [bq, bk, bv] if self.own_kv else [bq]
         self.w_in = torch.cat(ws, dim=0).contiguous()
@@ -480,19 +489,28 @@ class RotaryAttention:
             lam = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum())) + self.diff
             self.combine = (lam, self.eps, 1.0 - self.diff)
 
-    def context(self, h, batch, lc, dtype, out=None):
+    def context(self, h, batch, lc, dtype, out=None, y=None, carry=None):
         """The concatenated heads [T, heads * vdim] in front of W_o (into ``out`` if given); ``lc``: this layer's cache view, whose
-        pages are the lender's when keys and values are borrowed."""
+        pages are the lender's when keys and values are borrowed.  ``y``: the 32-bit projection by ``w_in``, if it is there already
+        (columns behind [q | k | v] are not this mixer's).  ``carry``: what one layer of a step leaves for later ones."""
         H, G, D, Dv = self.heads, self.kv_heads, self.dim, self.vdim
-        with trace("gemm_in"):
-            y = ops.linear(h, self.w_in, self.b_in, out_dtype=F32)
+        if y is None:
+            with trace("gemm_in"):
+                y = ops.linear(h, self.w_in, self.b_in, out_dtype=F32)
+        v_first = None
+        if self.v_mix == "first":
+            lo = (H + G) * self.maps * D
+            carry["v_first"] = y[:, lo:lo + G * Dv]
+        elif self.v_mix == "later":
+            v_first = carry["v_first"]
         with trace("norm_rope_kv_write"):
             q = ops.norm_rope_kv_write(y, H, G if self.own_kv else 0, D, Dv, self.maps, self.q_norm, self.k_norm, self.eps, self.freq,
                                        self.mag, self.interleaved, batch.positions, batch.slot_mapping, lc.k, lc.v, batch=batch,
-                                       scale=self.scale, out_dtype=dtype)
-        with trace("attention_window" if self.diff is None else "attention_diff"):
+                                       scale=self.scale, out_dtype=dtype, v_first=v_first, v_lam=self.v_lam)
+        with trace("attention_chunk" if self.chunk else "attention_window" if self.diff is None else "attention_diff"):
             return ops.attention_bias(q, lc.k, lc.v, batch, H, G, D, Dv, self.scale, None, out_dtype=dtype, window=self.window,
-                                      keep_first=self.keep_first, softcap=self.softcap, diff=self.combine, out=out)
+                                      keep_first=self.keep_first, softcap=self.softcap, diff=self.combine, out=out, chunk=self.chunk,
+                                      sinks=self.sinks)
 
     def forward(self, h, batch, lc, dtype):
         ctx = self.context(h, batch, lc, dtype)
@@ -665,34 +683,76 @@ class GatedFFN:
 
 
 class ParallelBlock:
-    """mixer(h) + ffn(h) as one sub-layer: W_o and W_down lie side by side, the mixer's heads and the feed-forward's hidden row
-    are written side by side, and one GEMM forms the sum of both outputs in 32-bit.  ``ffn`` None: the mixer alone.  The mixer
-    offers ``context(h, batch, lc, dtype, out)`` / ``n_out`` / ``w_o`` / ``b_o`` and the feed-forward ``hidden(h, out)`` / ``n_out`` /
-    ``w_down``."""
+    """mixer(h) + ffn(h) + experts(h) as one sub-layer, summed in 32-bit.  ``ffn`` (a GatedFFN: every token) and ``experts`` (a
+    blocks.RoutedExperts: each token its chosen few) may be None.
 
-    def __init__(self, mixer, ffn=None):
-        self.mixer, self.ffn = mixer, ffn
-        self.w_out = None
+    W_o and W_down (and the experts' down matrices) lie side by side; the mixer's heads and the hidden rows are written side by side,
+    and one GEMM forms the sum of all outputs in its accumulator.  With experts, the router's rows join the mixer's input
+    projection, and in the experts' dense form (RoutedExperts.form) one gated GEMM computes the hidden rows of ``ffn`` and of every
+    expert; in the other forms the chosen experts are added to the output product's result.
+
+    The mixer offers ``w_in`` / ``b_in`` and ``context(h, batch, lc, dtype, out, y, carry)`` / ``n_out`` / ``w_o`` / ``b_o``, the feed-forward
+    ``hidden(h, out)`` / ``n_out`` / ``w_gu`` / ``w_down``."""
+
+    def __init__(self, mixer, ffn=None, experts=None):
+        self.mixer, self.ffn, self.experts = mixer, ffn, experts
+        self.w_out = self.w_gu = None
 
     def weights(self):
-        """Both output matrices live in ``w_out`` after ``finalize``."""
-        m = [t for t in self.mixer.weights() if t is not self.mixer.w_o]
-        f = [t for t in self.ffn.weights() if t is not self.ffn.w_down] if self.ffn is not None else []
-        return m + f + [self.w_out]
+        """All output matrices live in ``w_out`` after ``finalize``, with experts all gate / up rows in ``w_gu`` and the router in the
+        mixer's ``w_in``."""
+        mx, ff, ex = self.mixer, self.ffn, self.experts
+        m = [t for t in mx.weights() if t is not mx.w_o and (ex is None or t is not mx.b_in)]
+        f = [t for t in ff.weights() if t is not ff.w_down and ex is None] if ff is not None else []
+        return m + f + [self.w_out] + ([self.w_gu, ex.b_router] if ex is not None else [])
 
     def finalize(self):
-        mx, ff = self.mixer, self.ffn
+        mx, ff, ex = self.mixer, self.ffn, self.experts
         self.n_ctx, self.n_cat = mx.n_out, mx.n_out + (ff.n_out if ff is not None else 0)
-        self.w_out = torch.cat([mx.w_o, ff.w_down], dim=1).contiguous() if ff is not None else mx.w_o
+        parts = [mx.w_o] + ([ff.w_down] if ff is not None else []) + ([ex.w_down] if ex is not None else [])
+        self.w_out = torch.cat(parts, dim=1).contiguous() if len(parts) > 1 else mx.w_o
         mx.w_o = self.w_out[:, :self.n_ctx]
         if ff is not None:
-            ff.w_down = self.w_out[:, self.n_ctx:]
+            ff.w_down = self.w_out[:, self.n_ctx:self.n_cat]
+        if ex is None:
+            return
+        ex.w_down = self.w_out[:, self.n_cat:]
+        assert ex.gated and (ff is None or ff.act == ex.act), "parallel block: experts and feed-forward share one gated product"
+        rows = ex.w_up.reshape(-1, ex.w_up.shape[-1])
+        self.w_gu = torch.cat([ff.w_gu, rows], dim=0).contiguous() if ff is not None else rows.contiguous()
+        n = 2 * ff.n_out if ff is not None else 0
+        if ff is not None:
+            ff.w_gu = self.w_gu[:n]
+        ex.w_up = self.w_gu[n:].view(ex.w_up.shape)
+        # the router reads the same input: its rows (and bias) behind the mixer's
+        w, b = mx.w_in, mx.b_in
+        if b is None:
+            b = torch.zeros(w.shape[0], dtype=w.dtype, device=w.device)
+        rb = ex.b_router if ex.b_router is not None else torch.zeros(ex.experts, dtype=w.dtype, device=w.device)
+        mx.w_in, mx.b_in = torch.cat([w, ex.in_rows()], dim=0).contiguous(), torch.cat([b, rb.to(w.dtype)]).contiguous()
+        self.n_in = ex.bind(w.shape[0])
 
-    def forward(self, h, batch, lc, dtype):
+    def forward(self, h, batch, lc, dtype, carry=None):
+        mx, ff, ex = self.mixer, self.ffn, self.experts
         T = h.shape[0]
-        cat = torch.empty(T, self.n_cat, dtype=dtype, device=h.device)
-        self.mixer.context(h, batch, lc, dtype, out=cat[:, :self.n_ctx])
-        if self.ffn is not None:
-            self.ffn.hidden(h, out=cat[:, self.n_ctx:])
+        y, form = None, None
+        if ex is not None:
+            form = ex.form(h)
+            # rows of a multiple of four numbers, whatever the expert count: 16-byte accesses for those who read them
+            y = torch.empty(T, -(-self.n_in // 4) * 4, dtype=F32, device=h.device)[:, :self.n_in]
+            with trace("gemm_in"):
+                ops.linear(h, mx.w_in, mx.b_in, out_dtype=F32, out=y)
+        dense = form == "dense"
+        cat = torch.empty(T, self.n_cat + (ex.n_hidden if dense else 0), dtype=dtype, device=h.device)
+        mx.context(h, batch, lc, dtype, out=cat[:, :self.n_ctx], y=y, carry=carry)
+        if dense:
+            with trace("ffn_up"):
+                ops.linear(h, self.w_gu, act=ex.act, gated=True, out=cat[:, self.n_ctx:])
+            ex.weigh(cat[:, self.n_cat:], y)
+        elif ff is not None:
+            ff.hidden(h, out=cat[:, self.n_ctx:])
         with trace("gemm_out"):
-            return ops.linear(cat, self.w_out, self.mixer.b_o, out_dtype=F32)
+            out = ops.linear(cat, self.w_out if dense or ex is None else self.w_out[:, :self.n_cat], mx.b_o, out_dtype=F32)
+        if ex is not None and not dense:
+            ex.forward(h, y, base=out, form=form)
+        return out

@@ -269,12 +269,13 @@ def moe_route(z, experts, top, groups, keep, route_scale, score="softmax", corre
     return ref.moe_route(z, experts, top, groups, keep, route_scale, score, correction, group_top, renorm)
 
 
-def moe_experts(h, ids, wts, w_up, w_down, act, gated: bool = False):
+def moe_experts(h, ids, wts, w_up, w_down, act, gated: bool = False, base=None):
+    """``base`` [T, W] 32-bit: the weighted sum is added to it in place."""
     if _cuda(h):
         from . import cuda_impl as cu
 
-        return cu.moe_experts(h, ids, wts, w_up, w_down, act, gated)
-    return ref.moe_experts(h, ids, wts, w_up, w_down, act, gated)
+        return cu.moe_experts(h, ids, wts, w_up, w_down, act, gated, base)
+    return ref.moe_experts(h, ids, wts, w_up, w_down, act, gated, base)
 
 
 # ----------------------------------------------------------------------------- recurrent layers, post-norm residual
@@ -314,20 +315,21 @@ def qknorm_kv_write(qkv, hq, hkv, dk, dv, q_w, k_w, eps, temp_coef, temp_every, 
 
 
 def attention_bias(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, dist_bias, gate=None, out_dtype=None, bias_over_scale=None,
-                   window=0, slopes=None, sinks=None, keep_first=0, softcap=0.0, diff=None, out=None):
+                   window=0, slopes=None, sinks=None, keep_first=0, softcap=0.0, diff=None, out=None, chunk=0):
     """Causal paged attention with separate key / value sizes, a per-head distance bias (a table, and / or a linear
     penalty ``slopes[h] * distance``), an optional sliding window, an output gate and an attention sink per head
     (``sinks`` [hq] 32-bit: exp(sinks[h]) joins every softmax denominator of head h).
     ``bias_over_scale``: dist_bias / scale, kept by the caller for the tensor-core kernels (derived per call if absent).
     ``keep_first``: first tokens that the window never hides; ``softcap``: cap * tanh(score / cap); ``diff`` = (lam, eps, factor): two
-    maps per head, combined as rms_div(a1 - lam * a2) * factor; ``out``: view that receives [T, hq * dv]."""
+    maps per head, combined as rms_div(a1 - lam * a2) * factor; ``out``: view that receives [T, hq * dv].
+    ``chunk``: keys outside the query's own block of ``chunk`` positions are hidden.  v_cache may be a column view of wider rows."""
     if _cuda(q):
         from . import cuda_impl as cu
 
         return cu.attention_bias(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, dist_bias, gate, out_dtype, bias_over_scale,
-                                 window, slopes, sinks, keep_first, softcap, diff, out)
+                                 window, slopes, sinks, keep_first, softcap, diff, out, chunk)
     return ref.attention_bias(q, k_cache, v_cache, batch.block_tables, batch.seq_lens, batch.cu_q, hq, hkv, dk, dv, scale,
-                              dist_bias, gate, out_dtype, window, slopes, sinks, keep_first, softcap, diff, out)
+                              dist_bias, gate, out_dtype, window, slopes, sinks, keep_first, softcap, diff, out, chunk)
 
 
 def unary(x, op, out_dtype=None):
@@ -377,16 +379,23 @@ def rope_norm_kv_write(qk, hq, hkv, d, freq, mag, interleaved, unit_norm, eps, p
 
 
 def latent_rope_prep(y, q_off, q_rank, c_off, rank, rot, g_off, n_gate, qn_w, cn_w, eps, freq, mag, positions, slot_mapping, cache,
-                     dtype):
+                     dtype, interleaved=True):
     """Normed query latent, normed key / value latent + rotated key part into the cache row, sigmoid gate columns."""
     return _dispatch("latent_rope_prep", y, y, q_off, q_rank, c_off, rank, rot, g_off, n_gate, qn_w, cn_w, eps, freq, mag, positions,
-                     slot_mapping, cache, dtype)
+                     slot_mapping, cache, dtype, interleaved)
 
 
-def latent_query_rope(q, heads, d, rot, rank, width, freq, mag, positions, dtype, abs_dtype):
+def latent_query_rope(q, heads, d, rot, rank, width, freq, mag, positions, dtype, abs_dtype, interleaved=True):
     """Split the up-projected queries into the unrotated operand of the absorption and the rotated part, placed in the
     absorbed-query buffer."""
-    return _dispatch("latent_query_rope", q, q, heads, d, rot, rank, width, freq, mag, positions, dtype, abs_dtype)
+    return _dispatch("latent_query_rope", q, q, heads, d, rot, rank, width, freq, mag, positions, dtype, abs_dtype, interleaved)
+
+
+def latent_rope_qkv(y, q_off, heads, d, c_off, rank, rot, cn_w, eps, freq, mag, interleaved, positions, slot_mapping, cache, dtype,
+                    abs_dtype):
+    """latent_rope_prep and latent_query_rope in one step where the queries are columns of the layer's own projection."""
+    return _dispatch("latent_rope_qkv", y, y, q_off, heads, d, c_off, rank, rot, cn_w, eps, freq, mag, interleaved, positions,
+                     slot_mapping, cache, dtype, abs_dtype)
 
 
 def hgrn_gates(y, n_qk, lower):
@@ -406,23 +415,23 @@ def softcap(z, cap):
     return _dispatch("softcap", z, z, cap)
 
 
-def residual_norm(resid, y, weight, bias, eps, kind, out_dtype=None):
-    """norm_residual over a 32-bit residual stream: (norm(resid + y) in ``out_dtype``, resid + y)."""
-    return _dispatch("residual_norm", resid, resid, y, weight, bias, eps, kind, out_dtype)
+def residual_norm(resid, y, weight, bias, eps, kind, out_dtype=None, mult=1.0):
+    """norm_residual over a 32-bit residual stream, r = resid + mult * y: (norm(r) in ``out_dtype``, r)."""
+    return _dispatch("residual_norm", resid, resid, y, weight, bias, eps, kind, out_dtype, mult)
 
 
 def norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, interleaved, positions, slot_mapping, k_cache, v_cache,
-                       batch=None, scale=1.0, out_dtype=None):
+                       batch=None, scale=1.0, out_dtype=None, v_first=None, v_lam=0.0):
     """Optional RMS norm with a weight per head (and map), rotation by a frequency table, keys and values to their pages; hkv = 0
-    prepares queries only.  ``batch`` and the score ``scale`` let the CUDA path lay the queries out for the attention kernel that will
+    prepares queries only.  ``v_first`` [T, hkv * dv] 32-bit: the values become (1 - v_lam) * v + v_lam * v_first.  ``batch`` and the score ``scale`` let the CUDA path lay the queries out for the attention kernel that will
     read them (attention_bias with the same ``batch``)."""
     if _cuda(qkv):
         from . import cuda_impl as cu
 
         return cu.norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, interleaved, positions, slot_mapping, k_cache,
-                                     v_cache, batch, scale, out_dtype)
+                                     v_cache, batch, scale, out_dtype, v_first, v_lam)
     return ref.norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, interleaved, positions, slot_mapping, k_cache,
-                                  v_cache, out_dtype)
+                                  v_cache, out_dtype, v_first, v_lam)
 
 
 def sample(logits, greedy, temperature, top_k, top_p, rng_state, vocab: Optional[int] = None, out=None):

@@ -190,6 +190,32 @@ _SIGS = {
     "llmss_attn_decode_span": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int64, c_void_p,
                                        c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_float,
                                        c_float, c_float, c_int, c_int, c_void_p]),
+    "llmss_residual_norm_ex": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                                       c_int, c_float, c_int, c_int, c_void_p]),
+    "llmss_norm_rope_kv_write_ex": (c_int, [c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
+                                            c_void_p, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                                            c_void_p, c_int, c_void_p, c_int64, c_float, c_int, c_int, c_void_p]),
+    "llmss_latent_rope_prep_ex": (c_int, [c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
+                                          c_float, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                                          c_void_p, c_int, c_int, c_void_p]),
+    "llmss_latent_query_rope_ex": (c_int, [c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_float, c_int,
+                                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "llmss_latent_rope_qkv": (c_int, [c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p,
+                                      c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+                                      c_int, c_void_p]),
+    "llmss_moe_experts_ex": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p,
+                                     c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "llmss_moe_combine_ex": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_void_p]),
+    "llmss_attention_span_ex": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p,
+                                        c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int,
+                                        c_int, c_int, c_int, c_int, c_float, c_int, c_void_p]),
+    "llmss_attn_prefill_span_ex": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
+                                           c_int64, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                                           c_float, c_int, c_int, c_int, c_float, c_void_p, c_float, c_float, c_float, c_int,
+                                           c_void_p]),
+    "llmss_attn_decode_span_ex": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
+                                          c_int64, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
+                                          c_int, c_int, c_float, c_void_p, c_float, c_float, c_float, c_int, c_int, c_void_p]),
     "llmss_gated_simt": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int,
                                  c_void_p]),
 }

@@ -590,18 +590,19 @@ def moe_route(z, experts, top, groups, keep, route_scale, dense: bool = False, s
     return (ids, wts, dn) if dense else (ids, wts)
 
 
-def moe_experts(h, ids, wts, w_up, w_down, act, gated: bool = False):
+def moe_experts(h, ids, wts, w_up, w_down, act, gated: bool = False, base=None):
     lib = _lib.load()
     T, W, ldh = _rows2d(h)
     E, F, _ = w_up.shape
     if gated:
         F //= 2       # rows interleave (gate_f, up_f)
     top = ids.shape[1]
-    assert w_up.is_contiguous() and w_down.is_contiguous() and h.dtype == w_up.dtype
+    assert w_up.is_contiguous() and w_down.stride(1) == 1 and h.dtype == w_up.dtype
     scratch = torch.empty(T, top, F, dtype=h.dtype, device=h.device)
-    out = torch.empty(T, W, dtype=torch.float32, device=h.device)
-    rc = lib.llmss_moe_experts(_ptr(h), ldh, _ptr(ids), _ptr(wts), _ptr(w_up), _ptr(w_down), w_down.stride(0), _ptr(scratch), _ptr(out),
-                               out.stride(0), T, W, F, top, act, 1 if gated else 0, _DT[h.dtype], _stream())
+    out = base if base is not None else torch.empty(T, W, dtype=torch.float32, device=h.device)
+    assert out.dtype == torch.float32 and out.shape == (T, W) and out.stride(1) == 1
+    rc = lib.llmss_moe_experts_ex(_ptr(h), ldh, _ptr(ids), _ptr(wts), _ptr(w_up), _ptr(w_down), w_down.stride(0), _ptr(scratch), _ptr(out),
+                                  out.stride(0), T, W, F, top, act, 1 if gated else 0, 0 if base is None else 1, _DT[h.dtype], _stream())
     _lib.check(rc, "llmss_moe_experts")
     _count(2)
     return out
@@ -615,7 +616,7 @@ def moe_scale(a, dense, experts: int, ff: int):
     return a
 
 
-def moe_experts_grouped(h, ids, wts, w_up, w_down, act, gated: bool = False):
+def moe_experts_grouped(h, ids, wts, w_up, w_down, act, gated: bool = False, base=None):
     """Long prompts: sort the (token, expert) pairs by expert on the device and run every expert as one pair of tensor-core
     GEMMs over its contiguous rows -- top / experts of the dense form's FLOPs.  Reads the per-expert counts on the host (one
     small synchronising copy), so it is for prompt processing, not for graph-captured decode steps."""
@@ -647,9 +648,10 @@ def moe_experts_grouped(h, ids, wts, w_up, w_down, act, gated: bool = False):
         if c:
             linear(xs[lo:lo + c], w_up[e], act=act, gated=gated, out=a[lo:lo + c])
             linear(a[lo:lo + c], w_down[:, e * F:(e + 1) * F], out_dtype=torch.float32, out=y[lo:lo + c])
-    out = torch.empty(T, W, dtype=torch.float32, device=dev)
-    _lib.check(lib.llmss_moe_combine(_ptr(y), _ptr(inv), _ptr(wts), _ptr(out), out.stride(0), T, W, top, _stream()),
-               "llmss_moe_combine")
+    out = base if base is not None else torch.empty(T, W, dtype=torch.float32, device=dev)
+    assert out.dtype == torch.float32 and out.shape == (T, W) and out.stride(1) == 1
+    _lib.check(lib.llmss_moe_combine_ex(_ptr(y), _ptr(inv), _ptr(wts), _ptr(out), out.stride(0), T, W, top, 0 if base is None else 1,
+                                        _stream()), "llmss_moe_combine")
     _count()
     return out
 
@@ -887,11 +889,14 @@ from .reference import window_bias_table  # noqa: E402  (the window and slopes a
 
 
 def attention_bias(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, dist_bias, gate=None, out_dtype=None, bias_over_scale=None,
-                   window=0, slopes=None, sinks=None, keep_first=0, softcap=0.0, diff=None, dst=None):
-    plain = dist_bias is None and slopes is None and gate is None and sinks is None
-    if plain or keep_first or softcap or diff is not None or dst is not None:
-        assert plain, "attention: kept first tokens, soft cap and two-map heads have no bias, slopes, gate or sink beside them"
-        return attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window or 0, keep_first, softcap, diff, out_dtype, dst)
+                   window=0, slopes=None, sinks=None, keep_first=0, softcap=0.0, diff=None, dst=None, chunk=0):
+    plain = dist_bias is None and slopes is None and gate is None
+    masked = (keep_first or softcap or diff is not None or dst is not None or chunk or not v_cache.is_contiguous()
+              or (sinks is not None and (window or dk != dv)))
+    if masked or (plain and sinks is None):
+        assert plain, "attention: span masks, soft cap, two-map heads and strided values have no bias, slopes or gate beside them"
+        return attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window or 0, keep_first, softcap, diff, out_dtype, dst,
+                              chunk, sinks)
     lib = _lib.load()
     T = q.shape[0]
     dt = q.dtype
@@ -998,52 +1003,76 @@ def span_decode_uses_tc(dtype, hq: int, hkv: int, dk: int, dv: int, maps: int, b
             and bool(_lib.load().llmss_attn_decode_tc_supported(hq * maps, hkv, _span_tile(dk, dv, maps), block_size)))
 
 
+def _span_decode_groups(dtype, hq: int, hkv: int, dk: int, dv: int, maps: int, block_size: int, scale: float):
+    """Head ranges of one tensor-core decode call each: all heads at once where the kernel's query tile holds a group; the heads
+    over one key / value head in groups of 32 or 8 where it does not; None where single tokens run on the prompt kernel."""
+    if span_decode_uses_tc(dtype, hq, hkv, dk, dv, maps, block_size, scale):
+        return [(0, hq)]
+    if hkv == 1 and maps == 1:
+        for n in (32, 8):
+            if n < hq and span_decode_uses_tc(dtype, n, 1, dk, dv, 1, block_size, scale):
+                return [(h, min(n, hq - h)) for h in range(0, hq, n)]
+    return None
+
+
 def attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window=0, keep_first=0, softcap=0.0, diff=None, out_dtype=None,
-                   out=None):
-    """attention_bias without additive terms; see ops.reference.attention_bias for window, keep_first, softcap and diff."""
+                   out=None, chunk=0, sinks=None):
+    """attention_bias without additive terms; see ops.reference.attention_bias for window, chunk, keep_first, softcap, diff, sinks and
+    values that are a column view of wider rows."""
     lib = _lib.load()
     T, dt, bs = q.shape[0], q.dtype, k_cache.shape[2]
     maps = 1 if diff is None else 2
-    assert k_cache.dtype == dt and (out_dtype or dt) == dt and q.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous()
-    assert k_cache.shape[1] == hkv and k_cache.shape[3] == maps * dk and v_cache.shape[3] == dv
+    ldv = v_cache.stride(2)
+    assert k_cache.dtype == dt and (out_dtype or dt) == dt and q.stride(1) == 1 and k_cache.is_contiguous()
+    assert k_cache.shape[1] == hkv and k_cache.shape[3] == maps * dk and v_cache.shape == (k_cache.shape[0], hkv, bs, dv)
+    assert v_cache.stride() == (hkv * bs * ldv, bs * ldv, ldv, 1), "attention: value pages are rows of one stride"
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == hq and sinks.is_contiguous() and maps == 1)
     if out is None:
         out = torch.empty(T, hq * dv, dtype=dt, device=q.device)
     assert out.dtype == dt and out.shape == (T, hq * dv) and out.stride(1) == 1
     lam, eps, factor = diff if diff is not None else (0.0, 0.0, 1.0)
-    if span_uses_tc(dt, dk, dv, maps, bs, scale):
+    if span_uses_tc(dt, dk, dv, maps, bs, scale) and ldv % 8 == 0:
         if out.stride(0) % 8 or out.data_ptr() % 16:     # a view whose rows miss the kernels' 16-byte stores
-            return out.copy_(attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window, keep_first, softcap, diff, out_dtype))
+            return out.copy_(attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window, keep_first, softcap, diff, out_dtype,
+                                            None, chunk, sinks))
         assert q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
-        if q.shape[1] == hq * maps * maps * dk and batch.is_decode and span_decode_uses_tc(dt, hq, hkv, dk, dv, maps, bs, scale):
+        groups = None
+        if q.shape[1] == hq * maps * maps * dk and batch.is_decode:
+            groups = _span_decode_groups(dt, hq, hkv, dk, dv, maps, bs, scale)
+        if groups is not None:
             d = _span_tile(dk, dv, maps)
-            reach = min(batch.max_kv, window + keep_first + 128) if window else batch.max_kv
-            splits = decode_splits(batch.num_seqs, hq * maps, hkv, d, reach, dt, bs)
-            scratch = None
-            if splits > 1 or maps == 2:
-                scratch = arena(q.device).attn_scratch(lib.llmss_attn_decode_scratch_floats(T, hq * maps, d, splits), q.device)
-            rc = lib.llmss_attn_decode_span(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables),
-                                            batch.block_tables.shape[1], _ptr(batch.seq_lens), _ptr(out), out.stride(0), _ptr(scratch), T,
-                                            hq, hkv, dk, dv, maps, bs, k_cache.shape[0], float(scale), int(window), int(keep_first),
-                                            float(softcap), float(lam), float(eps), float(factor), splits, _DT[dt], _stream())
-            _lib.check(rc, "llmss_attn_decode_span")
-            _count(1 if splits == 1 and maps == 1 else 2)
+            near = min(x for x in (window, chunk) if x) if window or chunk else 0
+            reach = min(batch.max_kv, near + keep_first + 128) if near else batch.max_kv
+            for h0, n in groups:
+                splits = decode_splits(batch.num_seqs, n * maps, hkv, d, reach, dt, bs)
+                scratch = None
+                if splits > 1 or maps == 2:
+                    scratch = arena(q.device).attn_scratch(lib.llmss_attn_decode_scratch_floats(T, n * maps, d, splits), q.device)
+                qv, ov = (q, out) if n == hq else (q[:, h0 * dk:(h0 + n) * dk], out[:, h0 * dv:(h0 + n) * dv])
+                rc = lib.llmss_attn_decode_span_ex(_ptr(qv), q.stride(0), _ptr(k_cache), _ptr(v_cache), ldv, _ptr(batch.block_tables),
+                                                   batch.block_tables.shape[1], _ptr(batch.seq_lens), _ptr(ov), out.stride(0), _ptr(scratch),
+                                                   T, n, hkv, dk, dv, maps, bs, k_cache.shape[0], float(scale), int(window), int(chunk),
+                                                   int(keep_first), float(softcap), _ptr(sinks[h0:h0 + n]) if sinks is not None else None,
+                                                   float(lam), float(eps), float(factor), splits, _DT[dt], _stream())
+                _lib.check(rc, "llmss_attn_decode_span")
+                _count(1 if splits == 1 and maps == 1 else 2)
             return out
         assert q.shape[1] == hq * maps * dk
-        rc = lib.llmss_attn_prefill_span(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables),
-                                         batch.block_tables.shape[1], _ptr(batch.seq_lens), _ptr(out), out.stride(0), _ptr(batch.cu_q),
-                                         batch.num_seqs, max(1, batch.max_q), T, hq, hkv, dk, dv, maps, bs, k_cache.shape[0], float(scale),
-                                         int(window), int(keep_first), float(softcap), float(lam), float(eps), float(factor), _DT[dt],
-                                         _stream())
+        rc = lib.llmss_attn_prefill_span_ex(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), ldv, _ptr(batch.block_tables),
+                                            batch.block_tables.shape[1], _ptr(batch.seq_lens), _ptr(out), out.stride(0), _ptr(batch.cu_q),
+                                            batch.num_seqs, max(1, batch.max_q), T, hq, hkv, dk, dv, maps, bs, k_cache.shape[0],
+                                            float(scale), int(window), int(chunk), int(keep_first), float(softcap), _ptr(sinks), float(lam),
+                                            float(eps), float(factor), _DT[dt], _stream())
         _lib.check(rc, "llmss_attn_prefill_span")
         _count()
         return out
     assert q.shape[1] == hq * maps * dk
     # the generic kernel: any sizes, true 32-bit; the two maps' outputs stay in 32-bit until they are combined
     o = torch.empty(T, hq * maps * dv, dtype=torch.float32, device=q.device) if maps == 2 else out
-    rc = lib.llmss_attention_span(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(batch.block_tables), batch.block_tables.shape[1],
-                                  bs, _ptr(batch.seq_lens), _ptr(batch.cu_q), int(window), int(keep_first), float(softcap), maps, _ptr(o),
-                                  o.stride(0), 1 if maps == 2 else 0, batch.num_seqs, max(1, batch.max_q), hq * maps, hkv, dk, dv,
-                                  float(scale), _DT[dt], _stream())
+    rc = lib.llmss_attention_span_ex(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), ldv, _ptr(batch.block_tables),
+                                     batch.block_tables.shape[1], bs, _ptr(batch.seq_lens), _ptr(batch.cu_q), int(window), int(chunk),
+                                     int(keep_first), float(softcap), maps, _ptr(sinks), _ptr(o), o.stride(0), 1 if maps == 2 else 0,
+                                     batch.num_seqs, max(1, batch.max_q), hq * maps, hkv, dk, dv, float(scale), _DT[dt], _stream())
     _lib.check(rc, "llmss_attention_span")
     _count()
     if maps == 2:
@@ -1053,7 +1082,7 @@ def attention_span(q, k_cache, v_cache, batch, hq, hkv, dk, dv, scale, window=0,
     return out
 
 
-def residual_norm(resid, y, weight, bias, eps, kind, out_dtype=None):
+def residual_norm(resid, y, weight, bias, eps, kind, out_dtype=None, mult=1.0):
     lib = _lib.load()
     T, W, ldr = _f32rows(resid)
     dt = out_dtype or torch.float32
@@ -1064,15 +1093,15 @@ def residual_norm(resid, y, weight, bias, eps, kind, out_dtype=None):
         assert Wy == W
     h = torch.empty(T, W, dtype=dt, device=resid.device)
     r = torch.empty(T, W, dtype=torch.float32, device=resid.device) if y is not None else resid
-    rc = lib.llmss_residual_norm(_ptr(resid), ldr, _ptr(y), ldy, _ptr(weight), _ptr(bias), _ptr(r) if y is not None else None, _ptr(h), T, W,
-                                 float(eps), int(kind), _DT[dt], _stream())
+    rc = lib.llmss_residual_norm_ex(_ptr(resid), ldr, _ptr(y), ldy, float(mult), _ptr(weight), _ptr(bias),
+                                    _ptr(r) if y is not None else None, _ptr(h), T, W, float(eps), int(kind), _DT[dt], _stream())
     _lib.check(rc, "llmss_residual_norm")
     _count()
     return h, r
 
 
 def norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, interleaved, positions, slot_mapping, k_cache, v_cache,
-                       batch=None, scale=1.0, out_dtype=None):
+                       batch=None, scale=1.0, out_dtype=None, v_first=None, v_lam=0.0):
     """``batch``: a batch of single tokens whose attention (score ``scale``) will run on the tensor-core decode kernel gets its queries
     as [T, hq * maps, maps * dk], zero outside the map's own columns."""
     lib = _lib.load()
@@ -1081,13 +1110,15 @@ def norm_rope_kv_write(qkv, hq, hkv, dk, dv, maps, q_w, k_w, eps, freq, mag, int
     assert k_cache.dtype == dt and v_cache.dtype == dt and k_cache.is_contiguous() and v_cache.is_contiguous()
     assert k_cache.shape[3] == maps * dk and (hkv == 0 or (k_cache.shape[1] == hkv and v_cache.shape[3] == dv))
     assert all(w is None or (w.dtype == torch.float32 and w.numel() == dk) for w in (q_w, k_w))
+    assert v_first is None or (v_first.dtype == torch.float32 and v_first.shape == (T, hkv * dv) and v_first.stride(1) == 1)
     hkv_pages, bs = k_cache.shape[1], k_cache.shape[2]      # (hkv = 0: the pages are another layer's)
     pad = int(maps > 1 and batch is not None and batch.is_decode
               and span_decode_uses_tc(dt, hq, hkv_pages, dk, v_cache.shape[3], maps, bs, scale))
     q = torch.empty(T, hq * maps * dk * (maps if pad else 1), dtype=dt, device=qkv.device)
-    rc = lib.llmss_norm_rope_kv_write(_ptr(qkv), ld, hq, hkv, dk, dv, maps, _ptr(q_w), _ptr(k_w), float(eps),
-                                      _ptr(_freq_dev(freq, qkv.device)), freq.numel(), float(mag), 1 if interleaved else 0, _ptr(positions),
-                                      _ptr(slot_mapping), _ptr(k_cache), _ptr(v_cache), k_cache.shape[2], _ptr(q), pad, T, _DT[dt], _stream())
+    rc = lib.llmss_norm_rope_kv_write_ex(_ptr(qkv), ld, hq, hkv, dk, dv, maps, _ptr(q_w), _ptr(k_w), float(eps),
+                                         _ptr(_freq_dev(freq, qkv.device)), freq.numel(), float(mag), 1 if interleaved else 0,
+                                         _ptr(positions), _ptr(slot_mapping), _ptr(k_cache), _ptr(v_cache), k_cache.shape[2], _ptr(q), pad,
+                                         _ptr(v_first), v_first.stride(0) if v_first is not None else 0, float(v_lam), T, _DT[dt], _stream())
     _lib.check(rc, "llmss_norm_rope_kv_write")
     _count()
     return q
@@ -1124,30 +1155,46 @@ def rope_norm_kv_write(qk, hq, hkv, d, freq, mag, interleaved, unit_norm, eps, p
     return q
 
 
-def latent_rope_prep(y, q_off, q_rank, c_off, rank, rot, g_off, n_gate, qn_w, cn_w, eps, freq, mag, positions, slot_mapping, cache, dtype):
+def latent_rope_prep(y, q_off, q_rank, c_off, rank, rot, g_off, n_gate, qn_w, cn_w, eps, freq, mag, positions, slot_mapping, cache, dtype,
+                     interleaved=True):
     lib = _lib.load()
     T, _, ldy = _f32rows(y)
     assert cache.dtype == dtype and cache.is_contiguous() and cn_w.dtype == torch.float32 and (q_rank == 0 or qn_w.dtype == torch.float32)
     cq = torch.empty(T, q_rank, dtype=dtype, device=y.device) if q_rank > 0 else None
     gate = torch.empty(T, n_gate, dtype=torch.float32, device=y.device) if n_gate > 0 else None
-    rc = lib.llmss_latent_rope_prep(_ptr(y), ldy, q_off, q_rank, c_off, rank, rot, g_off, n_gate, _ptr(qn_w), _ptr(cn_w), float(eps),
-                                    _ptr(_freq_dev(freq, y.device)), freq.numel(), float(mag), _ptr(positions), _ptr(slot_mapping),
-                                    _ptr(cache), cache.shape[-1], _ptr(cq), _ptr(gate), T, _DT[dtype], _stream())
+    rc = lib.llmss_latent_rope_prep_ex(_ptr(y), ldy, q_off, q_rank, c_off, rank, rot, g_off, n_gate, _ptr(qn_w), _ptr(cn_w), float(eps),
+                                       _ptr(_freq_dev(freq, y.device)), freq.numel(), float(mag), 1 if interleaved else 0, _ptr(positions),
+                                       _ptr(slot_mapping), _ptr(cache), cache.shape[-1], _ptr(cq), _ptr(gate), T, _DT[dtype], _stream())
     _lib.check(rc, "llmss_latent_rope_prep")
     _count()
     return cq, gate
 
 
-def latent_query_rope(q, heads, d, rot, rank, width, freq, mag, positions, dtype, abs_dtype):
+def latent_query_rope(q, heads, d, rot, rank, width, freq, mag, positions, dtype, abs_dtype, interleaved=True):
     lib = _lib.load()
     T, _, ldq = _f32rows(q)
     assert abs_dtype in (torch.float32, dtype)
     q_nope = torch.empty(T, heads * d, dtype=dtype, device=q.device)
     q_abs = torch.empty(T, heads * width, dtype=abs_dtype, device=q.device)
-    rc = lib.llmss_latent_query_rope(_ptr(q), ldq, heads, d, rot, rank, width, _ptr(_freq_dev(freq, q.device)), freq.numel(), float(mag),
-                                     _ptr(positions), _ptr(q_nope), _ptr(q_abs), 1 if abs_dtype == torch.float32 else 0, T, _DT[dtype],
-                                     _stream())
+    rc = lib.llmss_latent_query_rope_ex(_ptr(q), ldq, heads, d, rot, rank, width, _ptr(_freq_dev(freq, q.device)), freq.numel(), float(mag),
+                                        1 if interleaved else 0, _ptr(positions), _ptr(q_nope), _ptr(q_abs),
+                                        1 if abs_dtype == torch.float32 else 0, T, _DT[dtype], _stream())
     _lib.check(rc, "llmss_latent_query_rope")
+    _count()
+    return q_nope, q_abs
+
+
+def latent_rope_qkv(y, q_off, heads, d, c_off, rank, rot, cn_w, eps, freq, mag, interleaved, positions, slot_mapping, cache, dtype, abs_dtype):
+    lib = _lib.load()
+    T, _, ldy = _f32rows(y)
+    width = cache.shape[-1]
+    assert cache.dtype == dtype and cache.is_contiguous() and cn_w.dtype == torch.float32 and abs_dtype in (torch.float32, dtype)
+    q_nope = torch.empty(T, heads * d, dtype=dtype, device=y.device)
+    q_abs = torch.empty(T, heads * width, dtype=abs_dtype, device=y.device)
+    rc = lib.llmss_latent_rope_qkv(_ptr(y), ldy, q_off, heads, d, c_off, rank, rot, _ptr(cn_w), float(eps), _ptr(_freq_dev(freq, y.device)),
+                                   freq.numel(), float(mag), 1 if interleaved else 0, _ptr(positions), _ptr(slot_mapping), _ptr(cache),
+                                   width, _ptr(q_nope), _ptr(q_abs), 1 if abs_dtype == torch.float32 else 0, T, _DT[dtype], _stream())
+    _lib.check(rc, "llmss_latent_rope_qkv")
     _count()
     return q_nope, q_abs
 

@@ -274,10 +274,10 @@ def moe_route(z, experts: int, top: int, groups: int, keep: int, route_scale: fl
     return idx.to(torch.int32), w * route_scale
 
 
-def moe_experts(h, ids, wts, w_up, w_down, act: int, gated: bool = False):
+def moe_experts(h, ids, wts, w_up, w_down, act: int, gated: bool = False, base=None):
     """out[t] = sum_k wts[t, k] * W_down[ids[t, k]] act(W_up[ids[t, k]] h[t]);  w_up [E, F, W]; w_down [W, E * F] (the
     experts' down matrices side by side); fp32 result.  ``gated``: w_up is [E, 2 F, W] with rows interleaved (gate_0, up_0,
-    gate_1, ...) and the hidden activation is act(gate) * up."""
+    gate_1, ...) and the hidden activation is act(gate) * up.  ``base`` [T, W] 32-bit: the result is added to it in place."""
     T, W = h.shape
     E, F, _ = w_up.shape
     up = w_up.float()[ids.long()]                       # [T, top, F, W]
@@ -287,8 +287,9 @@ def moe_experts(h, ids, wts, w_up, w_down, act: int, gated: bool = False):
         a = (apply_act(a[..., 0::2], act) * a[..., 1::2]).to(h.dtype).float()
     else:
         a = apply_act(a, act).to(h.dtype).float()
-    down = w_down.float().view(W, E, F).permute(1, 0, 2)[ids.long()]   # [T, top, W, F]
-    return torch.einsum("tkwf,tkf,tk->tw", down, a, wts.float())
+    down = w_down.float().reshape(W, E, F).permute(1, 0, 2)[ids.long()]   # [T, top, W, F]
+    y = torch.einsum("tkwf,tkf,tk->tw", down, a, wts.float())
+    return y if base is None else base.add_(y)
 
 
 def _fmix32(x):
@@ -613,7 +614,7 @@ def window_bias_table(slopes, window: int, scale: float):
 
 def attention_bias(q, k_cache, v_cache, block_tables, seq_lens, cu_q, hq: int, hkv: int, dk: int, dv: int, scale: float,
                    dist_bias, gate=None, out_dtype=None, window: int = 0, slopes=None, sinks=None, keep_first: int = 0,
-                   softcap: float = 0.0, diff=None, out=None):
+                   softcap: float = 0.0, diff=None, out=None, chunk: int = 0):
     """Causal softmax attention over the paged cache with key size dk, value size dv, grouped heads, an additive bias
     dist_bias[h, min(i - j, last)] per head and distance (or none), a linear penalty slopes[h] * (i - j) taken off the
     scores (or none), a sliding window (``window`` > 0: query i sees keys j with 0 <= i - j < window), an optional
@@ -623,13 +624,15 @@ def attention_bias(q, k_cache, v_cache, block_tables, seq_lens, cu_q, hq: int, h
     visible.  ``softcap`` > 0: the scaled score s becomes softcap * tanh(s / softcap) before anything is added to it.
     ``diff`` = (lam, eps, factor): every head has two query / key maps of size dk over its one value (q [T, hq * 2 * dk], K pages
     [.., 2 * dk], map 1 first); with a1, a2 the maps' outputs the head's output is rms_div(a1 - lam * a2) * factor.
-    ``out``: [T, hq * dv] view that receives the result."""
+    ``chunk`` > 0: query i sees only keys of its own block of ``chunk`` positions (j // chunk = i // chunk, counted from the
+    sequence's start), the kept first tokens excepted.  ``out``: [T, hq * dv] view that receives the result.  v_cache may be a
+    column view of wider rows (latent attention: the leading columns of the key row are the value)."""
     if diff is not None:
         lam, eps, factor = diff
         nb, _, bs, dk2 = k_cache.shape
         halves = [attention_bias(q.reshape(-1, hq, 2, dk)[:, :, m].reshape(-1, hq * dk), k_cache[..., m * dk:(m + 1) * dk], v_cache,
                                  block_tables, seq_lens, cu_q, hq, hkv, dk, dv, scale, dist_bias, gate, torch.float32, window, slopes,
-                                 sinks, keep_first, softcap).view(-1, hq, dv) for m in (0, 1)]
+                                 sinks, keep_first, softcap, chunk=chunk).view(-1, hq, dv) for m in (0, 1)]
         o = (_rms_div(halves[0] - lam * halves[1], eps) * factor).reshape(-1, hq * dv).to(out_dtype or q.dtype)
         return o if out is None else out.copy_(o)
     T = q.shape[0]
@@ -659,6 +662,8 @@ def attention_bias(q, k_cache, v_cache, block_tables, seq_lens, cu_q, hq: int, h
         hidden = kpos > qpos
         if window > 0:
             hidden = hidden | ((qpos - kpos >= window) & (kpos >= keep_first))
+        if chunk > 0:
+            hidden = hidden | ((qpos // chunk != kpos // chunk) & (kpos >= keep_first))
         s = s.masked_fill(hidden, float("-inf"))
         if sinks is not None:
             p = torch.softmax(torch.cat([s, sinks.float().view(hq, 1, 1).expand(hq, ql, 1)], dim=-1), dim=-1)[..., :L]
@@ -876,11 +881,11 @@ def rope_norm_kv_write(qk, hq: int, hkv: int, d: int, freq, mag: float, interlea
 
 
 def latent_rope_prep(y, q_off: int, q_rank: int, c_off: int, rank: int, rot: int, g_off: int, n_gate: int, qn_w, cn_w, eps: float,
-                     freq, mag: float, positions, slot_mapping, cache, dtype):
+                     freq, mag: float, positions, slot_mapping, cache, dtype, interleaved: bool = True):
     """First stage of latent attention with a rotated key part, on the layer's fused 32-bit projection y [T, *]:
     the query latent y[:, q_off : q_off + q_rank] is RMS-normed (weight ``qn_w``) and returned in ``dtype`` (the operand of the
     query up-projection; q_rank = 0: there is none); the key / value latent y[:, c_off : c_off + rank] is RMS-normed
-    (weight ``cn_w``), the ``rot`` columns behind it are rotated (interleaved pairs) and not normed, and both are written
+    (weight ``cn_w``), the ``rot`` columns behind it are rotated (pairs (2i, 2i + 1) if ``interleaved`` else (i, i + n)) and not normed, and both are written
     side by side into the token's cache row (cache [num_blocks, block_size, >= rank + rot]; columns beyond are zeroed);
     sigmoid of the n_gate gate columns is returned in 32-bit ([T, n_gate], or None)."""
     T = y.shape[0]
@@ -888,7 +893,7 @@ def latent_rope_prep(y, q_off: int, q_rank: int, c_off: int, rank: int, rot: int
     if q_rank > 0:
         cq = (_rms_div(y[:, q_off:q_off + q_rank].float(), eps) * qn_w.float()).to(dtype)
     c = _rms_div(y[:, c_off:c_off + rank].float(), eps) * cn_w.float()
-    kr = _rotate_by_table(y[:, c_off + rank:c_off + rank + rot].float().reshape(T, 1, rot), positions, freq, mag, True).reshape(T, rot)
+    kr = _rotate_by_table(y[:, c_off + rank:c_off + rank + rot].float().reshape(T, 1, rot), positions, freq, mag, interleaved).reshape(T, rot)
     width = cache.shape[-1]
     row = torch.zeros(T, width, dtype=torch.float32, device=y.device)
     row[:, :rank], row[:, rank:rank + rot] = c, kr
@@ -898,16 +903,27 @@ def latent_rope_prep(y, q_off: int, q_rank: int, c_off: int, rank: int, rot: int
     return cq, gate
 
 
-def latent_query_rope(q, heads: int, d: int, rot: int, rank: int, width: int, freq, mag: float, positions, dtype, abs_dtype):
+def latent_query_rope(q, heads: int, d: int, rot: int, rank: int, width: int, freq, mag: float, positions, dtype, abs_dtype,
+                      interleaved: bool = True):
     """Second stage: q [T, heads * (d + rot)] (every head [d unrotated | rot rotated]).  Returns (q_nope [T, heads * d] in
     ``dtype`` -- the operand of the per-head key absorption -- and the absorbed-query buffer [T, heads * width] in
-    ``abs_dtype`` whose columns [rank, rank + rot) of every head hold the rotated part (interleaved pairs); columns below
+    ``abs_dtype`` whose columns [rank, rank + rot) of every head hold the rotated part (pairs as in latent_rope_prep); columns below
     ``rank`` are left for the absorption product, columns beyond rank + rot are zero."""
     T = q.shape[0]
-    qh = q.float().view(T, heads, d + rot)
+    qh = q.float().reshape(T, heads, d + rot)
     qa = torch.zeros(T, heads, width, dtype=abs_dtype, device=q.device)
-    qa[:, :, rank:rank + rot] = _rotate_by_table(qh[..., d:], positions, freq, mag, True).to(abs_dtype)
+    qa[:, :, rank:rank + rot] = _rotate_by_table(qh[..., d:], positions, freq, mag, interleaved).to(abs_dtype)
     return qh[..., :d].reshape(T, heads * d).to(dtype), qa.view(T, heads * width)
+
+
+def latent_rope_qkv(y, q_off: int, heads: int, d: int, c_off: int, rank: int, rot: int, cn_w, eps: float, freq, mag: float,
+                    interleaved: bool, positions, slot_mapping, cache, dtype, abs_dtype):
+    """Both stages at once for latent attention whose queries come straight from the layer's projection y [T, *] (no query
+    latent, no gate): y[:, q_off : q_off + heads * (d + rot)] as in latent_query_rope, y[:, c_off : c_off + rank + rot] as in
+    latent_rope_prep.  Returns (q_nope, absorbed-query buffer)."""
+    latent_rope_prep(y, 0, 0, c_off, rank, rot, 0, 0, None, cn_w, eps, freq, mag, positions, slot_mapping, cache, dtype, interleaved)
+    return latent_query_rope(y[:, q_off:q_off + heads * (d + rot)], heads, d, rot, rank, cache.shape[-1], freq, mag, positions, dtype,
+                             abs_dtype, interleaved)
 
 
 def hgrn_gates(y, n_qk: int, lower):
@@ -947,9 +963,11 @@ def softcap(z, cap: float):
 
 
 # ----------------------------------------------------------------------------- norms over a 32-bit residual, normed and rotated q / k
-def residual_norm(resid, y, weight, bias, eps: float, kind: int, out_dtype=None):
-    """norm_residual over a 32-bit residual stream: r = resid + y (y None: r = resid), h = LayerNorm or RMS norm of r.
+def residual_norm(resid, y, weight, bias, eps: float, kind: int, out_dtype=None, mult: float = 1.0):
+    """norm_residual over a 32-bit residual stream: r = resid + mult * y (y None: r = resid), h = LayerNorm or RMS norm of r.
     Returns (h in ``out_dtype``, r 32-bit)."""
+    if y is not None and mult != 1.0:
+        y = y.float() * mult
     h, r = norm_residual(resid, y, weight, bias if kind == NORM_LAYER else None, eps, kind, out_dtype=torch.float32)
     if bias is not None and kind != NORM_LAYER:
         h = h + bias.float()
@@ -957,12 +975,13 @@ def residual_norm(resid, y, weight, bias, eps: float, kind: int, out_dtype=None)
 
 
 def norm_rope_kv_write(qkv, hq: int, hkv: int, dk: int, dv: int, maps: int, q_w, k_w, eps: float, freq, mag: float, interleaved: bool,
-                       positions, slot_mapping, k_cache, v_cache, out_dtype=None):
+                       positions, slot_mapping, k_cache, v_cache, out_dtype=None, v_first=None, v_lam: float = 0.0):
     """Queries, keys and values of grouped-query attention from the fused 32-bit projection qkv [T, hq*maps*dk | hkv*maps*dk |
     hkv*dv].  Every head has ``maps`` query / key vectors of size dk, side by side.  Each is divided by its root mean square and
     multiplied by the weight q_w / k_w [dk] (None: no norm), then rotated by the frequency table; keys go to the K pages
     [blocks, hkv, block_size, maps * dk], the values as they are to the V pages.  hkv = 0: queries only (a layer that attends
-    over another layer's pages).  Returns the queries [T, hq * maps * dk]."""
+    over another layer's pages).  ``v_first`` [T, hkv*dv] 32-bit (another layer's values of the same tokens): the pages take
+    (1 - v_lam) * v + v_lam * v_first.  Returns the queries [T, hq * maps * dk]."""
     T = qkv.shape[0]
 
     def prepare(x, w):
@@ -976,6 +995,8 @@ def norm_rope_kv_write(qkv, hq: int, hkv: int, dk: int, dv: int, maps: int, q_w,
         lo = (hq + hkv) * maps * dk
         k = prepare(qkv[:, hq * maps * dk:lo].reshape(T, hkv * maps, dk), k_w).reshape(T, hkv, maps * dk)
         v = qkv[:, lo:lo + hkv * dv].reshape(T, hkv, dv)
+        if v_first is not None:
+            v = (1.0 - v_lam) * v.float() + v_lam * v_first.float().reshape(T, hkv, dv)
         bs = k_cache.shape[2]
         valid = slot_mapping >= 0
         slots = slot_mapping[valid].long()

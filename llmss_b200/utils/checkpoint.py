@@ -546,6 +546,89 @@ PRESETS.update({
 })
 
 
+def fipavik_config(width: int, vocab: int, layers, residual_mult: float = 1.0, eps: float = 1e-6) -> dict:
+    """config.json of a Fipavik model.  ``layers``: one dict per layer,
+    {"type": "latent_attention", heads, dim, rot_dim, vdim, kv_rank, window} | {"type": "attention", heads, kv_heads, dim, vdim, chunk,
+    optionally rot_dims, v_mix}, each optionally with base, scale, and with "mlp": None | {"experts", "top", "ff", "shared"} (``shared``: the
+    hidden size of the expert every token takes, or None)."""
+    out = []
+    for L in layers:
+        latent = L["type"] == "latent_attention"
+        span = L["rot_dim"] if latent else L["dim"]
+        m = {k: L[k] for k in ("heads", "dim", "vdim") + (("rot_dim", "kv_rank") if latent else ("kv_heads",))}
+        m.update(rot={"base": L.get("base", 10000.0), "dims": span if latent else L.get("rot_dims", span)},
+                 scale=L.get("scale", (L["dim"] + L["rot_dim"] if latent else L["dim"]) ** -0.5),
+                 mask={"size": L["window"] if latent else L["chunk"]})
+        if not latent:
+            m["v_mix"] = bool(L.get("v_mix", True))
+        f = L.get("mlp")
+        mlp = None
+        if f is not None:
+            mlp = {"kind": "moe", "expert": {"ff": f["ff"]}, "router": {"experts": f["experts"], "top": f["top"]}}
+            if f.get("shared") is not None:
+                mlp["shared"] = {"ff": f["shared"]}
+        out.append({"type": L["type"], "mixer": m, "mlp": mlp})
+    return {"architecture": "Fipavik", "vocab": vocab, "width": width, "norm": {"eps": eps}, "residual_mult": residual_mult, "layers": out}
+
+
+def _fipavik_shapes(cfg: dict):
+    W, V = cfg["width"], cfg["vocab"]
+    yield "embed", (V, W), ("n", 0.0, 1.0)
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}", L["mixer"]
+        q, H, d, dv = f"{p}.mix", m["heads"], m["dim"], m["vdim"]
+        yield f"{p}.norm1", (W,), "ln_w"
+        yield f"{p}.norm1.b", (W,), ("n", 0.0, 0.1)
+        if L["type"] == "latent_attention":
+            r, R = m["rot_dim"], m["kv_rank"]
+            yield f"{q}.q", (H * (d + r), W), "fan"
+            yield f"{q}.dkv", (R + r, W), "fan"
+            yield f"{q}.dkv.norm", (R,), "ln_w"
+            yield f"{q}.uk", (H * d, R), "fan"
+            yield f"{q}.uv", (H * dv, R), "fan"
+        else:
+            G = m["kv_heads"]
+            for s, n in (("q", H * d), ("k", G * d), ("v", G * dv)):
+                yield f"{q}.{s}", (n, W), "fan"
+            for s in ("q", "k"):
+                yield f"{q}.{s}.norm", (d,), "ln_w"
+            if m.get("v_mix"):
+                yield f"{q}.vmix", (), ("u", 0.2, 0.6)
+        yield f"{q}.sink", (H,), ("n", 0.0, 1.0)
+        yield f"{q}.o", (W, H * dv), "fan"
+        f = L.get("mlp")
+        if f is None:
+            continue
+        E, F = f["router"]["experts"], f["expert"]["ff"]
+        yield f"{p}.mlp.router", (E, W), "fan2"
+        yield f"{p}.mlp.router.b", (E,), ("n", 0.0, 0.2)
+        for e, n in [(f"e{e}", F) for e in range(E)] + ([("shared", f["shared"]["ff"])] if f.get("shared") is not None else []):
+            yield f"{p}.mlp.{e}.gate", (n, W), "fan2"
+            yield f"{p}.mlp.{e}.up", (n, W), "fan"
+            yield f"{p}.mlp.{e}.down", (W, n), "fan2"
+    yield "final.norm", (W,), "ln_w"
+    yield "final.norm.b", (W,), ("n", 0.0, 0.1)
+
+
+def _fipavik_preset(width, vocab, heads, ff, shared, experts, top, n_blocks, rank=192, window=1024, chunk=2048):
+    """n_blocks x (windowed latent attention, two chunked attention layers), experts everywhere."""
+    mlp = dict(experts=experts, top=top, ff=ff, shared=shared)
+    lat = dict(type="latent_attention", heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=rank, window=window, mlp=mlp)
+    att = dict(type="attention", heads=heads, kv_heads=max(1, heads // 4), dim=128, vdim=128, rot_dims=64, chunk=chunk, base=500000.0, mlp=mlp)
+    return fipavik_config(width, vocab, [dict(L) for _ in range(n_blocks) for L in (lat, att, att)], residual_mult=0.5)
+
+
+PRESETS.update({
+    "fipavik-tiny": fipavik_config(128, 320, [
+        dict(type="attention", heads=4, kv_heads=2, dim=24, vdim=40, rot_dims=16, chunk=20, mlp=dict(experts=6, top=2, ff=48, shared=64)),
+        dict(type="latent_attention", heads=6, dim=24, rot_dim=16, vdim=32, kv_rank=40, window=33, mlp=dict(experts=4, top=3, ff=32, shared=40)),
+        dict(type="attention", heads=4, kv_heads=2, dim=32, vdim=40, rot_dims=8, chunk=48, mlp=None)], residual_mult=0.6),
+    # sizes whose layers resemble a served model's (random weights), beside gptj-like-* and zenorax-* of equal width and depth
+    "fipavik-2k": _fipavik_preset(2048, 32000, 16, 1024, 1024, 16, 4, 6),
+    "fipavik-4k": _fipavik_preset(4096, 32000, 32, 1536, 2048, 32, 4, 6),
+})
+
+
 def _shapes(cfg: dict) -> Iterator[Tuple[str, Tuple[int, ...], str]]:
     """(name, shape, kind) for every tensor of the family; kind in {w, b, ln_w, ln_b, emb} (and, for architectures whose
     activations must keep unit scale without trained weights: unit, fan, fan2, alpha, ls)."""
@@ -560,6 +643,8 @@ def _shapes(cfg: dict) -> Iterator[Tuple[str, Tuple[int, ...], str]]:
         yield from _zenorax_shapes(cfg)
     elif mt == "rofulorn":
         yield from _rofulorn_shapes(cfg)
+    elif mt == "fipavik":
+        yield from _fipavik_shapes(cfg)
     elif mt == "gptj":
         H, L, V = cfg["n_embd"], cfg["n_layer"], cfg["vocab_size"]
         F = cfg.get("n_inner") or 4 * H
