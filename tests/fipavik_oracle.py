@@ -95,11 +95,9 @@ def expert(h, p, pre):
 
 def route(z, top):
     """z [T, E] logits -> [T, E] weights: softmax over the ``top`` largest, 0 elsewhere."""
-    w = torch.zeros_like(z)
-    for t in range(z.shape[0]):
-        ids = sorted(range(z.shape[1]), key=lambda e: (-z[t, e].item(), e))[:top]
-        w[t, ids] = torch.softmax(z[t, ids], dim=-1)
-    return w
+    chosen = torch.sort(z, dim=-1, descending=True, stable=True).indices[:, :top]
+    e = torch.exp(z.gather(1, chosen) - z.max(-1, keepdim=True).values)
+    return torch.zeros_like(z).scatter(1, chosen, e / e.sum(-1, keepdim=True))
 
 
 def mixture(h, p, pre, f):
