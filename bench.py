@@ -55,7 +55,7 @@ def parse():
     ap.add_argument("--compare", default=None, metavar="A:B[,A:B...]",
                     help="instead of the headline run: prefill and decode tokens/s plus per-op device times of preset A beside "
                          "preset B (e.g. bedovik-2k:gptj-like-2k, ninelix-2k:gptj-like-2k, botalorn-2k:gptj-like-2k, zenorax-2k:gptj-like-2k, "
-                         "rofulorn-2k:gptj-like-2k), "
+                         "rofulorn-2k:gptj-like-2k, fipavik-2k:zenorax-2k), "
                          "one JSON line per preset")
     return ap.parse_args()
 

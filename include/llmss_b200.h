@@ -432,6 +432,53 @@ int llmss_attn_decode_span(const void* q, int64_t ldq, const void* k_cache, cons
                            int max_blocks, const int* seq_lens, void* out, int64_t ldo, float* scratch, int B, int hq, int hkv, int dk,
                            int dv, int maps, int block_size, int num_blocks, float scale, int window, int keep_first, float cap,
                            float lam, float eps, float factor, int num_splits, int dtype, llmss_stream_t stream);
+/* ---- chunked masks, sinks and strided values in the span kernels; value mixing; latent attention without a query latent; experts
+ * added to another product */
+/* llmss_residual_norm with a factor on y: out_r = resid + mult * y */
+int llmss_residual_norm_ex(const float* resid, int64_t ldr, const float* y, int64_t ldy, float mult, const float* weight,
+                           const float* bias, float* out_r, void* out_h, int M, int W, float eps, int kind, int out_dtype,
+                           llmss_stream_t stream);
+/* llmss_norm_rope_kv_write with v_first [T][hkv*dv] 32-bit (row stride ldf, or null): the V pages take (1 - v_lam) v + v_lam v_first */
+int llmss_norm_rope_kv_write_ex(const float* qkv, int64_t ld, int hq, int hkv, int dk, int dv, int maps, const float* q_w,
+                                const float* k_w, float eps, const double* freq, int n_pairs, float mag, int interleaved,
+                                const int* positions, const int* slots, void* k_cache, void* v_cache, int block_size, void* q_out,
+                                int pad, const float* v_first, int64_t ldf, float v_lam, int T, int dtype, llmss_stream_t stream);
+/* the span kernels with a chunked mask (chunk > 0: a query sees its own block of `chunk` positions, counted from the sequence's
+ * start), a sink logit per head (sinks [hq] 32-bit or null; maps = 1) and V pages whose rows are ldv >= dv numbers apart (latent
+ * attention: v_cache = k_cache, the leading dv columns of the key row are the value; the tcgen05 forms want ldv a multiple of 8) */
+int llmss_attention_span_ex(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, int ldv, const int* block_tables,
+                            int max_blocks, int block_size, const int* seq_lens, const int* cu_q, int window, int chunk,
+                            int keep_first, float cap, int maps, const float* sinks, void* out, int64_t ldo, int out_f32, int B,
+                            int max_q, int hq, int hkv, int dk, int dv, float scale, int dtype, llmss_stream_t stream);
+int llmss_attn_prefill_span_ex(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, int ldv, const int* block_tables,
+                               int max_blocks, const int* seq_lens, void* out, int64_t ldo, const int* cu_q, int num_seqs, int max_q,
+                               int total_q, int hq, int hkv, int dk, int dv, int maps, int block_size, int num_blocks, float scale,
+                               int window, int chunk, int keep_first, float cap, const float* sinks, float lam, float eps,
+                               float factor, int dtype, llmss_stream_t stream);
+int llmss_attn_decode_span_ex(const void* q, int64_t ldq, const void* k_cache, const void* v_cache, int ldv, const int* block_tables,
+                              int max_blocks, const int* seq_lens, void* out, int64_t ldo, float* scratch, int B, int hq, int hkv,
+                              int dk, int dv, int maps, int block_size, int num_blocks, float scale, int window, int chunk,
+                              int keep_first, float cap, const float* sinks, float lam, float eps, float factor, int num_splits,
+                              int dtype, llmss_stream_t stream);
+/* llmss_latent_rope_prep / _query_rope with a choice of pairs (interleaved: (2i, 2i+1), else (i, i + n_pairs)), and both in one step
+ * where the queries [H * (d + rot)] are columns of y from q_off on and [latent (rank) | key part (rot)] lie from c_off on */
+int llmss_latent_rope_prep_ex(const float* y, int64_t ldy, int q_off, int q_rank, int c_off, int rank, int rot, int g_off, int n_gate,
+                              const float* qn_w, const float* cn_w, float eps, const double* freq, int n_pairs, float mag,
+                              int interleaved, const int* positions, const int* slots, void* cache, int width, void* cq_out,
+                              float* gate, int T, int dtype, llmss_stream_t stream);
+int llmss_latent_query_rope_ex(const float* q, int64_t ldq, int H, int d, int rot, int rank, int width, const double* freq,
+                               int n_pairs, float mag, int interleaved, const int* positions, void* q_nope, void* q_abs, int abs_f32,
+                               int T, int dtype, llmss_stream_t stream);
+int llmss_latent_rope_qkv(const float* y, int64_t ldy, int q_off, int H, int d, int c_off, int rank, int rot, const float* cn_w,
+                          float eps, const double* freq, int n_pairs, float mag, int interleaved, const int* positions,
+                          const int* slots, void* cache, int width, void* q_nope, void* q_abs, int abs_f32, int T, int dtype,
+                          llmss_stream_t stream);
+/* llmss_moe_experts / _combine with add = 1: the weighted sum is added to out */
+int llmss_moe_experts_ex(const void* h, int64_t ldh, const int* ids, const float* wts, const void* w_up, const void* w_down,
+                         int64_t ldd, void* act_scratch, float* out, int64_t ldo, int T, int W, int F, int top, int act, int gated,
+                         int add, int dtype, llmss_stream_t stream);
+int llmss_moe_combine_ex(const float* y, const int* inv, const float* wts, float* out, int64_t ldo, int T, int W, int top, int add,
+                         llmss_stream_t stream);
 /* out[t][n] = act(x_t . w_2n) * (x_t . w_2n+1) on the CUDA cores (any size, 32-bit or 16-bit) */
 int llmss_gated_simt(const void* x, int64_t ldx, const void* w, int64_t ldw, const void* bias, void* out, int64_t ldo, int M,
                      int n_out, int K, int act, int dtype, llmss_stream_t stream);
