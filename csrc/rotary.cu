@@ -132,8 +132,8 @@ __global__ void __launch_bounds__(256) rope_norm_kv_write_kernel(const float* __
 
 // norm_rope_kv_write: block 256, a warp per vector of the token's row (hq * maps queries, hkv * maps keys, hkv values).  Grid
 // (T, S): a decode batch spreads a token's vectors over S blocks, a prompt keeps them in one.  Vector form (sizes that are
-// multiples of four; pairs (2i, 2i + 1), or (i, i + n) with n a multiple of four, whose partner columns are read again through
-// L1): LPV lanes share a vector (16: short ones, two per warp) and hold NV 4-column groups each in
+// multiples of four; pairs (2i, 2i + 1), or (i, i + n) with n a multiple of four, whose partner columns come from the lane that
+// holds them, or for long vectors are read again through L1): LPV lanes share a vector (16: short ones, two per warp) and hold NV 4-column groups each in
 // registers from the 16-byte load to the store; the next P vectors are loaded before the first is worked on.  NV = 0: element
 // by element, any size.
 struct NrArgs {
@@ -182,21 +182,18 @@ __device__ __forceinline__ const float* nr_source(const NrArgs& a, int64_t t, in
 
 template <typename T, int NV, int LPV>
 __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
-  __shared__ float cs[kMaxPairs], sn[kMaxPairs];
+  __shared__ __align__(16) float cs[kMaxPairs], sn[kMaxPairs];
   const int64_t t = blockIdx.x;
-  pdl_launch_dependents();
-  token_angles(a.freq, a.n, a.positions[t], a.mag, cs, sn);      // inputs of the step, not of the kernel in front
-  pdl_wait();
-  __syncthreads();
   const int warp = blockIdx.y * 8 + (threadIdx.x >> 5), warps = gridDim.y * 8, lane = threadIdx.x & 31;
   const int dk = a.dk, nu = a.hq * a.maps + a.hkv * (a.maps + 1);
-  const int slot = a.hkv > 0 ? a.slots[t] : -1;
+  pdl_launch_dependents();
+  const int slot = a.hkv > 0 ? a.slots[t] : -1;                  // this and the angles: inputs of the step, not of the kernel in front
   if constexpr (NV > 0) {
     constexpr int P = NV <= 2 ? 4 / NV : 1, VPW = 32 / LPV;
     const int sub = lane / LPV, l4 = (lane % LPV) * 4, step = warps * VPW;
     const uint32_t mates = LPV == 32 ? 0xffffffffu : (uint32_t)((1u << (LPV & 31)) - 1u) << (sub * LPV);
-    for (int u0 = warp * VPW + sub; u0 < nu; u0 += step * P) {
-      float v[P][NV > 0 ? NV : 1][4];
+    float v[P][NV > 0 ? NV : 1][4];
+    auto fetch = [&](int u0) {
 #pragma unroll
       for (int p = 0; p < P; ++p) {
         const int u = u0 + p * step;
@@ -211,6 +208,13 @@ __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
           v[p][i][0] = f.x; v[p][i][1] = f.y; v[p][i][2] = f.z; v[p][i][3] = f.w;
         }
       }
+    };
+    pdl_wait();
+    fetch(warp * VPW + sub);                                     // in flight while the angles are formed
+    token_angles(a.freq, a.n, a.positions[t], a.mag, cs, sn);
+    __syncthreads();
+    for (int u0 = warp * VPW + sub; u0 < nu; u0 += step * P) {
+      if (u0 != warp * VPW + sub) fetch(u0);
 #pragma unroll
       for (int p = 0; p < P; ++p) {
         const int u = u0 + p * step;
@@ -233,33 +237,42 @@ __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
           const int c = l4 + i * (LPV * 4);
-          if (c >= width) continue;
-          if (w != nullptr) {
+          if (w != nullptr && c < width) {
             const float4 wv = *reinterpret_cast<const float4*>(w + c);
             v[p][i][0] *= rstd * wv.x; v[p][i][1] *= rstd * wv.y; v[p][i][2] *= rstd * wv.z; v[p][i][3] *= rstd * wv.w;
           }
-          if (map >= 0 && !a.interleaved) {
-            if (c < 2 * a.n) {
-              const bool second = c >= a.n;
-              const int pc = second ? c - a.n : c + a.n, p0 = second ? pc : c;       // partner column, first pair of the group
-              float4 o = *reinterpret_cast<const float4*>(nr_source(a, t, u) + pc);
+          if (map >= 0 && !a.interleaved && a.n > 0) {
+            const bool turns = c < 2 * a.n, second = c >= a.n;
+            const int pc = !turns ? c : second ? c - a.n : c + a.n, p0 = second ? pc : c;       // partner column, first pair of the group
+            float ov[4];
+            if constexpr (NV == 1) {                             // all lanes of the vector take part
+#pragma unroll
+              for (int e = 0; e < 4; ++e) ov[e] = __shfl_sync(mates, v[p][i][e], pc >> 2, LPV);
+            } else if (turns) {
+              const float4 o = *reinterpret_cast<const float4*>(nr_source(a, t, u) + pc);
+              ov[0] = o.x; ov[1] = o.y; ov[2] = o.z; ov[3] = o.w;
               if (w != nullptr) {
                 const float4 wv = *reinterpret_cast<const float4*>(w + pc);
-                o.x *= rstd * wv.x; o.y *= rstd * wv.y; o.z *= rstd * wv.z; o.w *= rstd * wv.w;
-              }
-              const float ov[4] = {o.x, o.y, o.z, o.w};
-#pragma unroll
-              for (int e = 0; e < 4; ++e) {
-                const float so = ov[e] * sn[p0 + e];
-                v[p][i][e] = fmaf(v[p][i][e], cs[p0 + e], second ? so : -so);
+                ov[0] *= rstd * wv.x; ov[1] *= rstd * wv.y; ov[2] *= rstd * wv.z; ov[3] *= rstd * wv.w;
               }
             }
-          } else if (map < 0 && a.v_first != nullptr) {
+            if (turns) {
+              const float4 cc = *reinterpret_cast<const float4*>(cs + p0), ss = *reinterpret_cast<const float4*>(sn + p0);
+              const float cv[4] = {cc.x, cc.y, cc.z, cc.w}, sv[4] = {ss.x, ss.y, ss.z, ss.w};
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const float so = ov[e] * sv[e];
+                v[p][i][e] = fmaf(v[p][i][e], cv[e], second ? so : -so);
+              }
+            }
+          }
+          if (c >= width) continue;
+          if (map < 0 && a.v_first != nullptr) {
             const float4 f = *reinterpret_cast<const float4*>(a.v_first + t * a.ldf + (int64_t)(u - (nu - a.hkv)) * a.dv + c);
             const float fv[4] = {f.x, f.y, f.z, f.w};
 #pragma unroll
             for (int e = 0; e < 4; ++e) v[p][i][e] = fmaf(1.f - a.v_lam, v[p][i][e], a.v_lam * fv[e]);
-          } else if (map >= 0) {
+          } else if (map >= 0 && a.interleaved) {
 #pragma unroll
             for (int e = 0; e < 4; e += 2) {
               const int pr = (c + e) >> 1;
@@ -281,6 +294,9 @@ __global__ void __launch_bounds__(256) norm_rope_kv_write_kernel(NrArgs a) {
       }
     }
   } else {
+    token_angles(a.freq, a.n, a.positions[t], a.mag, cs, sn);
+    pdl_wait();
+    __syncthreads();
     for (int u = warp; u < nu; u += warps) {
       int width, map;
       const float* w;
